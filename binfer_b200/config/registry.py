@@ -75,6 +75,8 @@ def _register_builtin() -> None:
     register_architecture("Ketopel", KetopelConfig.from_dict)
     from .folivik import FolivikConfig
     register_architecture("Folivik", FolivikConfig.from_dict)
+    from .pabelix import PabelixConfig
+    register_architecture("Pabelix", PabelixConfig.from_dict)
 
 
 _register_builtin()

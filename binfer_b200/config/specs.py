@@ -121,12 +121,19 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """Dense gated feed-forward: down(act(gate(x)) * up(x))."""
+    """Dense gated feed-forward: down(act(gate(x)) * up(x)).
+
+    ``activation`` "clamped": with ``g = min(gate(x), limit)`` and ``u = clamp(up(x), -limit,
+    limit)`` the product is ``g sigmoid(slope g) (u + up_offset)``."""
 
     kind: str = "gated_mlp"
     intermediate_size: int = 0
     activation: str = "silu"     # or "gelu_tanh": 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+                                 # or "clamped"
     bias: bool = False
+    limit: float = 0.0           # "clamped" only, like the two below
+    slope: float = 1.0
+    up_offset: float = 0.0
     # the tensors' names inside the feed-forward's prefix: gate, up, down
     names: Tuple[str, str, str] = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
 
@@ -306,6 +313,45 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Grouped-query causal softmax attention in which a head is the difference of two maps.
+    A query head and a key head hold two vectors of ``head_dim`` each, one per map; both maps
+    weigh the same values of ``value_dim``.  With a1 and a2 their outputs::
+
+        lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + diff
+        o = a1 - lambda a2;   o <- o / sqrt(mean(o^2) + norm_eps) (1 - diff)
+
+    (the mean over the head's values; the four vectors have ``head_dim`` numbers, and lambda
+    is one number for the layer).  Scores are ``(q . k) scale``; no rotation.
+
+    ``temp_coef``, ``temp_every``: q at position p is multiplied by ``1 + temp_coef ln(floor((p
+    + 1) / temp_every) + 1)`` (``temp_coef`` 0: not).  ``output_gate``: the concatenated heads
+    are multiplied element by element by the sigmoid of a projection of the mixer's input.
+    ``own_cache`` False: the layer reads another layer's keys and values and has no key or
+    value tensors of its own.  ``names``: the tensors inside the mixer's prefix."""
+
+    kind: str = "differential_attention"
+    num_heads: int = 0
+    num_kv_heads: int = 0
+    head_dim: int = 0            # of one map
+    value_dim: int = 0
+    scale: Optional[float] = None    # None = 1/sqrt(head_dim)
+    diff: float = 0.0
+    norm_eps: float = 1e-6
+    temp_coef: float = 0.0
+    temp_every: int = 1
+    output_gate: bool = True
+    own_cache: bool = True
+    names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("k", "k"), ("v", "v"), ("g", "g"),
+                                          ("o", "o"), ("lq1", "lq1"), ("lk1", "lk1"),
+                                          ("lq2", "lq2"), ("lk2", "lk2"))
+
+    @property
+    def softmax_scale(self) -> float:
+        return self.scale if self.scale is not None else self.head_dim ** -0.5
+
+
+@dataclass(frozen=True)
 class GatedDeltaRuleSpec:
     """A matrix memory written by the delta rule with a decay per token and head.  Per value
     head, with a state ``S [qk_dim, v_dim]`` that starts at zero::
@@ -398,7 +444,12 @@ class MoESpec:
     outputs form that many equal groups of neighbours, a group counts by its largest choice
     score, and only the outputs of the best ``groups_keep`` groups can be chosen.
     ``identity`` > 0: the router has that many outputs behind the experts' that stand for
-    experts whose output is their input (no tensors)."""
+    experts whose output is their input (no tensors).
+
+    ``scoring`` "sigmoid": the scores are the sigmoids of the router outputs, each on its own;
+    everything else as for "softmax_all".  ``group_top``: a group counts by the sum of its
+    that many largest choice scores.  ``normalize`` False: the chosen scores are not divided
+    by their sum."""
 
     kind: str = "moe"
     num_experts: int = 0
@@ -420,6 +471,8 @@ class MoESpec:
     groups: int = 1
     groups_keep: int = 1
     identity: int = 0
+    group_top: int = 1
+    normalize: bool = True
 
 
 @dataclass(frozen=True)
@@ -431,8 +484,9 @@ class LayerSpec:
                                  # arrangement has no second sublayer in this layer)
     norm: NormSpec = NormSpec()
     block: str = "prenorm"       # arrangement of the parts inside the layer: "prenorm",
-                                 # "sublayer_norm", or "parallel" (one norm, both sublayers
-                                 # read it, their sum is added)
+                                 # "sublayer_norm", "parallel" (one norm, both sublayers
+                                 # read it, their sum is added), or "sandwich" (a norm before
+                                 # and one after each sublayer)
 
 
 @dataclass(frozen=True)
@@ -462,6 +516,14 @@ class ScheduleEntry:
 
 
 @dataclass(frozen=True)
+class PositionVectorSpec:
+    """A sinusoidal vector per position, added to the embedding output: at position p entry
+    2i is ``sin(p base^(-2i / hidden_size))`` and entry 2i + 1 the cosine of the same."""
+
+    base: float = 10000.0
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     architecture: str
     hidden_size: int
@@ -482,6 +544,8 @@ class ModelSpec:
     # (tensor name, rows) of a table ``[rows, hidden_size]`` whose rows schedule entries add
     # to the stream (ScheduleEntry.before); None: the model has none
     pass_table: Optional[Tuple[str, int]] = None
+    # added to the embedding output; None: nothing (positions enter in the mixers only)
+    position_vectors: Optional[PositionVectorSpec] = None
 
 
 @dataclass(frozen=True)

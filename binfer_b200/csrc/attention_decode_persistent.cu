@@ -22,6 +22,14 @@
 // the pool's scratch page, so a slot never holds stale bits, and a masked probability of
 // zero always meets a finite V.  (The cache pool is allocated zeroed.)
 //
+// The same kernel as a template instance (PAIR) runs differential attention: a cached key row
+// holds the keys of two maps side by side (64 or 128 columns each), a query head two vectors
+// of that size, one per map, and both maps weigh the same values.  The tile's row 2h + m is
+// map m of head h; its query is zero in the other map's columns, which the fragments supply
+// as zeros, so K and V are fetched once for both maps.  nh then counts rows (two a head), a
+// row of scores has a factor that grows with the query's position, and the partial results go
+// to the merge kernel that also makes the two maps one (attention_diff.cu).
+//
 // Takes head sizes 64, 128, 256, page sizes that divide 128 and are at least 8, up to 16
 // query heads per kv head and up to DP_MAX_ROWS rows; the caller uses the second kernel for
 // everything else.  All waits are bounded (about a second): the thread that gives up sets
@@ -30,6 +38,7 @@
 #include <float.h>
 #include <stdlib.h>
 
+#include "attention_diff.cuh"
 #include "common.cuh"
 #include "mma_utils.cuh"
 #include "tma_utils.cuh"
@@ -141,7 +150,7 @@ __device__ __forceinline__ DpItem dp_lookup(int idx, bool lane_on, int first, in
   return d;
 }
 
-template <int D>
+template <int D, bool PAIR>
 __global__ void __launch_bounds__(DP_THREADS, 1)
 decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
                                    const __grid_constant__ CUtensorMap map_v,
@@ -156,7 +165,8 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
                                    int n_rows, int nh, int nkv, int page_size, int num_pages,
                                    int window, int max_splits, float scale_log2, int slots,
                                    int groups, int early, int* __restrict__ err, float cap_pre,
-                                   float cap_post) {
+                                   float cap_post, long long q_stride, float temp_coef,
+                                   int temp_every) {
   constexpr int HALVES = D / 64;
   constexpr int HALF_ELEMS = DP_SPLIT * 64;
   constexpr int TILE_ELEMS = DP_SPLIT * D;
@@ -164,12 +174,13 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
   extern __shared__ __align__(16) unsigned char smem_raw[];
   unsigned char* base = smem_raw + ((1024u - (bf_smem_u32(smem_raw) & 1023u)) & 1023u);
   const int G = nh / nkv;
+  const int GQ = PAIR ? G / 2 : G;                       // query vectors of D numbers per kv head
   // Each consumer group has a ring of its own (spg slots, qsg query buffers): a slot is
   // then filled and read by the same parties in strict turn, which the one-bit phase of an
   // mbarrier needs.  (Were a slot shared, the group that reads its next fill could ask for
   // that phase while the fill before it is still in flight, and the parity would say yes.)
   const int spg = slots / groups, qsg = (spg + 1) / 2;
-  const DpSmem L = dp_layout(D, slots, groups, G, n_rows);
+  const DpSmem L = dp_layout(D, slots, groups, GQ, n_rows);
   __nv_bfloat16* tiles = reinterpret_cast<__nv_bfloat16*>(base);
   uint64_t* full = reinterpret_cast<uint64_t*>(base + L.bars);
   uint64_t* empty = full + DP_MAX_SLOTS;
@@ -260,9 +271,9 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
           int* inf = info + e * 8;
           if (inf[7]) {
             inf[7] = 0;
-            dp_bulk_load(qbuf + (size_t)e * G * D,
-                         q + ((size_t)inf[5] * nh + (size_t)inf[1] * G) * D,
-                         (uint32_t)(G * D * 2), full + inf[6]);
+            dp_bulk_load(qbuf + (size_t)e * GQ * D,
+                         q + (size_t)inf[5] * q_stride + (size_t)inf[1] * GQ * D,
+                         (uint32_t)(GQ * D * 2), full + inf[6]);
           }
         }
       __syncwarp();
@@ -315,10 +326,11 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
             const int t = row_t[r];
             int* inf = info + qi * 8;
             inf[0] = r; inf[1] = g; inf[2] = split;
-            bf_mbar_expect_tx(full + slot, TILE_BYTES + (uint32_t)(G * D * 2));
+            bf_mbar_expect_tx(full + slot, TILE_BYTES + (uint32_t)(GQ * D * 2));
             if (waited) {
-              dp_bulk_load(qbuf + (size_t)qi * G * D, q + ((size_t)t * nh + (size_t)g * G) * D,
-                           (uint32_t)(G * D * 2), full + slot);
+              dp_bulk_load(qbuf + (size_t)qi * GQ * D,
+                           q + (size_t)t * q_stride + (size_t)g * GQ * D,
+                           (uint32_t)(GQ * D * 2), full + slot);
             } else {
               inf[5] = t; inf[6] = slot; inf[7] = 1;
             }
@@ -389,15 +401,18 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
 
     unsigned qa[D / 16][4];
     {
-      const __nv_bfloat16* q0 = qbuf + (size_t)qi * G * D + (size_t)r0 * D;
-      const __nv_bfloat16* q1 = q0 + (size_t)8 * D;
+      // (PAIR: rows 2h and 2h + 1 share a query row, each sees its own half of the columns)
+      const __nv_bfloat16* q0 = qbuf + (size_t)qi * GQ * D + (size_t)(PAIR ? r0 >> 1 : r0) * D;
+      const __nv_bfloat16* q1 = q0 + (size_t)(PAIR ? 4 : 8) * D;
 #pragma unroll
       for (int ks = 0; ks < D / 16; ++ks) {
         const int c = ks * 16 + cq;
-        qa[ks][0] = r0 < G ? *reinterpret_cast<const unsigned*>(q0 + c) : 0u;
-        qa[ks][1] = r0 + 8 < G ? *reinterpret_cast<const unsigned*>(q1 + c) : 0u;
-        qa[ks][2] = r0 < G ? *reinterpret_cast<const unsigned*>(q0 + c + 8) : 0u;
-        qa[ks][3] = r0 + 8 < G ? *reinterpret_cast<const unsigned*>(q1 + c + 8) : 0u;
+        const bool mine = !PAIR || (r0 & 1) == (ks >= D / 32 ? 1 : 0);
+        const bool lo = mine && r0 < G, hi = mine && r0 + 8 < G;
+        qa[ks][0] = lo ? *reinterpret_cast<const unsigned*>(q0 + c) : 0u;
+        qa[ks][1] = hi ? *reinterpret_cast<const unsigned*>(q1 + c) : 0u;
+        qa[ks][2] = lo ? *reinterpret_cast<const unsigned*>(q0 + c + 8) : 0u;
+        qa[ks][3] = hi ? *reinterpret_cast<const unsigned*>(q1 + c + 8) : 0u;
       }
     }
     float s[4][4];
@@ -418,7 +433,7 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
     __syncwarp();
     if (lane == 0) dp_mbar_arrive(empty + slotK);        // K tile, queries and info are in registers
 
-    if (cap_pre > 0.f) {       // s <- (c / scale) tanh(s scale / c): the scale still rides below
+    if (!PAIR && cap_pre > 0.f) {       // s <- (c / scale) tanh(s scale / c): the scale still rides below
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
@@ -430,12 +445,14 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
       }
     }
     float m0 = -INFINITY, m1 = -INFINITY;
+    float sc = scale_log2;
+    if (PAIR) sc *= bf_query_temperature(p, temp_coef, temp_every);
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int j = k_begin + wkey + nt * 8 + cq + (i & 1);
-        s[nt][i] = (j >= j0 && j <= p) ? s[nt][i] * scale_log2 : -INFINITY;
+        s[nt][i] = (j >= j0 && j <= p) ? s[nt][i] * sc : -INFINITY;
       }
       m0 = fmaxf(m0, fmaxf(s[nt][0], s[nt][1]));
       m1 = fmaxf(m1, fmaxf(s[nt][2], s[nt][3]));
@@ -545,14 +562,15 @@ static int dp_sm_count() {
   return counts[dev];
 }
 
-template <int D>
+template <int D, bool PAIR = false>
 static int launch_persistent(const void* q, const void* k_cache, const void* v_cache,
                              const int* rows, const int* seq_of_token, const int* positions,
                              const int* block_tables, int table_stride, float* part_o,
                              float* part_ml, int n_rows, int nh, int nkv, int page_size,
                              int num_pages, int window, int max_splits, float scale, int* err,
-                             cudaStream_t stream, float softcap) {
-  const int G = nh / nkv;
+                             cudaStream_t stream, float softcap, long long q_stride,
+                             float temp_coef = 0.f, int temp_every = 1) {
+  const int G = nh / nkv / (PAIR ? 2 : 1);
   const size_t limit = 227 * 1024;
   int slots = DP_MAX_SLOTS;
   int groups = DP_GROUPS;
@@ -576,7 +594,7 @@ static int launch_persistent(const void* q, const void* k_cache, const void* v_c
   e = bf_make_tensor_map_pages_bf16(&mvr, v_cache, num_pages, nkv, page_size, D,
                                     DP_SPLIT / page_size);
   if (e) return e;
-  auto kern = decode_attention_persistent_kernel<D>;
+  auto kern = decode_attention_persistent_kernel<D, PAIR>;
   static bool configured_on[BF_MAX_DEVICES];
   bool& configured = configured_on[bf_current_device()];
   if (!configured) {
@@ -595,7 +613,7 @@ static int launch_persistent(const void* q, const void* k_cache, const void* v_c
                        window, max_splits, scale * 1.4426950408889634f, slots, groups,
                        getenv("BINFER_B200_ATTN_EARLY") ? atoi(getenv("BINFER_B200_ATTN_EARLY")) : 1,
                        err, softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f,
-                       softcap > 0.f ? softcap / scale : 0.f);
+                       softcap > 0.f ? softcap / scale : 0.f, q_stride, temp_coef, temp_every);
 }
 
 // The arguments and result of bf_decode_attention, and: a soft cap c > 0 on the scaled
@@ -621,7 +639,7 @@ BF_EXPORT int bf_decode_attention_persistent_capped(
     e = launch_persistent<DD>(q, k_cache, v_cache, rows, seq_of_token, positions,            \
                               block_tables, table_stride, part_o, part_ml, n_rows, nh, nkv,  \
                               page_size, num_pages, window, max_splits, scale, err, stream,  \
-                              softcap);                                                      \
+                              softcap, (long long)nh * d);                                   \
     break
   switch (d) {
     DP_CASE(64);
@@ -649,6 +667,45 @@ BF_EXPORT int bf_decode_attention_persistent(const void* q, const void* k_cache,
       q, k_cache, v_cache, rows, seq_of_token, positions, block_tables, table_stride, out,
       part_o, part_ml, n_rows, nh, nkv, d, page_size, num_pages, window, max_splits, scale, err,
       0.f, (long long)nh * d, 1.f, stream);
+}
+
+// Differential attention of single tokens: nh heads of two maps with d / 2 key columns each (a
+// cached key row holds both, d) over values of d; d 64, 128 or 256, at most 8 heads per kv head.
+// q: rows `q_stride` elements apart, head h at columns h d.  part_o [n_rows, nh, 2, max_splits, d],
+// part_ml likewise; the rest as above and in attention_diff.cuh.
+BF_EXPORT int bf_diff_attention_decode_persistent(
+    const void* q, long long q_stride, const void* k_cache, const void* v_cache, const int* rows,
+    const int* seq_of_token, const int* positions, const int* block_tables, int table_stride,
+    void* out, float* part_o, float* part_ml, int n_rows, int nh, int nkv, int d, int page_size,
+    int num_pages, int max_splits, float scale, int* err, long long out_stride, const void* gate,
+    long long gate_stride, float lambda, float eps, float out_factor, float temp_coef,
+    int temp_every, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (nkv <= 0 || nh % nkv || nh / nkv > 8 || n_rows > DP_MAX_ROWS || page_size < 8 ||
+      page_size > 128 || DP_SPLIT % page_size || ((uintptr_t)k_cache & 15) ||
+      ((uintptr_t)v_cache & 15) || ((uintptr_t)q & 15) || (q_stride & 7) ||
+      q_stride < (long long)nh * d || !(scale > 0.f) || temp_every < 1 || temp_coef < 0.f)
+    return (int)cudaErrorInvalidValue;
+  int e;
+#define DP_PAIR_CASE(DD)                                                                     \
+  case DD:                                                                                   \
+    e = launch_persistent<DD, true>(q, k_cache, v_cache, rows, seq_of_token, positions,      \
+                                    block_tables, table_stride, part_o, part_ml, n_rows,     \
+                                    2 * nh, nkv, page_size, num_pages, 0, max_splits, scale, \
+                                    err, stream, 0.f, q_stride, temp_coef, temp_every);      \
+    break
+  switch (d) {
+    DP_PAIR_CASE(64);
+    DP_PAIR_CASE(128);
+    DP_PAIR_CASE(256);
+    default:
+      return (int)cudaErrorInvalidValue;
+  }
+#undef DP_PAIR_CASE
+  if (e) return e;
+  const BfDiffArgs dd = {gate, gate_stride, lambda, eps, out_factor, temp_coef, temp_every};
+  return bf_diff_attention_merge_rows(part_o, part_ml, rows, positions, out, n_rows, nh, d,
+                                      max_splits, out_stride, dd, stream);
 }
 
 BF_TRACE_READER(bf_trace_read_attention_decode_persistent)

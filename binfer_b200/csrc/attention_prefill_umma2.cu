@@ -32,6 +32,16 @@
 // has no rows runs with group B idle.  Head size 128 only; the caller takes the first
 // arrangement for head size 64 and for portions of at most 128 queries.
 //
+// The same kernel as a template instance (DIFF) runs differential attention with two maps of
+// 64 key columns over values of 128: the two query tiles are then the two maps of the SAME
+// 128 queries and one head.  A cached key row holds both maps' keys side by side, so the two
+// 64-column halves that a K tile is staged in anyway are the two maps' K tiles, and V is
+// shared: one fetch of K and V serves both maps.  Each query row may have a factor on its
+// scores that grows with its position.  The epilogue makes the two maps one: every softmax
+// warp reads 32 columns of BOTH O tiles of its rows from tensor memory, forms a1 - lambda a2,
+// the four warps of a quarter exchange their sums of squares, and the normed head leaves
+// multiplied by its gate.
+//
 // Every mbarrier wait is bounded.  A barrier whose waiter could fall two phases behind exists
 // once per parity of the tile number, so that its one-bit phase cannot alias: "P V of tile n
 // done" (waited for only when O must be rescaled), and "P of tile n written" (a softmax
@@ -43,6 +53,7 @@
 #include <float.h>
 #include <stdint.h>
 
+#include "attention_diff.cuh"
 #include "common.cuh"
 #include "tma_utils.cuh"
 #include "umma_utils.cuh"
@@ -57,20 +68,23 @@ constexpr int A2_TMA_WARP = 16;
 constexpr int A2_MMA_WARP = 17;  // 17 issues for query tile A, 18 for tile B
 constexpr int A2_D = 128;
 
-// Barrier among the 256 softmax threads of a group that also ANDs a predicate.
+// Barrier among the 256 softmax threads of a group (or THREADS of both) that also ANDs a
+// predicate.
+template <int THREADS = 256>
 __device__ __forceinline__ bool group_all(int id, bool ok) {
   uint32_t r;
   asm volatile(
       "{\n\t.reg .pred p, q;\n\t"
       "setp.ne.b32 q, %1, 0;\n\t"
-      "barrier.cta.red.and.pred p, %2, 256, q;\n\t"
+      "barrier.cta.red.and.pred p, %2, %3, q;\n\t"
       "selp.b32 %0, 1, 0, p;\n\t}"
       : "=r"(r)
-      : "r"((uint32_t)ok), "r"(id)
+      : "r"((uint32_t)ok), "r"(id), "n"(THREADS)
       : "memory");
   return r != 0;
 }
 
+template <bool DIFF>
 __global__ void __launch_bounds__(A2_THREADS, 1)
 prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
                                const __grid_constant__ CUtensorMap map_k,
@@ -83,9 +97,11 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
                                int num_pages, int window, float scale_log2, int splits,
                                float* __restrict__ part_o, float* __restrict__ part_ml,
                                int* __restrict__ err, float cap_pre, float cap_post,
-                               long long out_stride, float out_scale) {
+                               long long out_stride, float out_scale, BfDiffArgs dd) {
   constexpr int D = A2_D;
   constexpr int HALVES = D / 64;
+  constexpr int BROWS = DIFF ? A2_BM : 2 * A2_BM;        // query rows of a CTA
+  constexpr int TSHIFT = DIFF ? 0 : A2_BM;               // rows from query tile A to tile B
   constexpr int QHALF_BYTES = A2_BM * 128;               // 128 query rows of 128 bytes
   constexpr int KHALF_BYTES = A2_BN * 128;               // 64 key rows of 128 bytes
   constexpr int Q_BYTES = HALVES * QHALF_BYTES;          // one Q tile
@@ -97,7 +113,8 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
   uint8_t* Ks = Qs + 2 * Q_BYTES;                        // [STAGES][KV_BYTES]
   uint8_t* Vs = Ks + A2_STAGES * KV_BYTES;               // [STAGES][KV_BYTES]
   float* xm = reinterpret_cast<float*>(Vs + A2_STAGES * KV_BYTES);   // [sums, references][2 groups][128]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(xm + 4 * 128);
+  float* xss = xm + 4 * 128;                             // DIFF: [4 column quarters][128] sums of squares
+  uint64_t* bars = reinterpret_cast<uint64_t*>(xss + (DIFF ? 4 * 128 : 0));
   uint64_t* q_full = bars;                     // [1]
   uint64_t* kv_full = bars + 1;                // [STAGES]
   uint64_t* kv_empty = kv_full + A2_STAGES;    // [STAGES]
@@ -117,16 +134,16 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
   // portion start first and the short ones fill in behind them (with the query block in x a
   // long block could start late and end alone: 80 us for 2048 tokens from position 0).
   const int qb = (int)gridDim.z - 1 - (int)blockIdx.z, h = blockIdx.x;
-  if (qb * 2 * A2_BM >= qlen) return;
-  const bool active_b = qb * 2 * A2_BM + A2_BM < qlen;
+  if (qb * BROWS >= qlen) return;
+  const bool active_b = DIFF || qb * BROWS + A2_BM < qlen;
   const int g = h / (nh / nkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int* table = block_tables + (size_t)seq * table_stride;
   const int pages = A2_BN / page_size;
 
-  const int p_first = pos0 + qb * 2 * A2_BM;                            // first row of tile A
+  const int p_first = pos0 + qb * BROWS;                                // first row of tile A
   const int p_last_a = min(pos0 + qlen - 1, p_first + A2_BM - 1);
-  const int p_last = active_b ? min(pos0 + qlen - 1, p_first + 2 * A2_BM - 1) : p_last_a;
+  const int p_last = active_b ? min(pos0 + qlen - 1, p_first + BROWS - 1) : p_last_a;
   const int j_lo = window > 0 ? max(0, p_first - window + 1) : 0;
   int kt_first = j_lo / A2_BN;
   int tiles_a = p_last_a / A2_BN - kt_first + 1;
@@ -169,13 +186,20 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
   if (warp == A2_TMA_WARP) {
     // ---------------------------------------------------------------- TMA producer
     if (lane == 0 && tiles > 0) {                        // (a share of the keys may be empty)
-      mbar_expect_tx(q_full, 2 * Q_BYTES);
+      if constexpr (DIFF) {                              // 64 columns of each map
+        mbar_expect_tx(q_full, 2 * QHALF_BYTES);
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+        for (int t = 0; t < 2; ++t)
+          tma_load_2d(Qs + t * Q_BYTES, &map_q, q_full, h * D + t * 64, row0 + qb * BROWS);
+      } else {
+        mbar_expect_tx(q_full, 2 * Q_BYTES);
 #pragma unroll
-        for (int hh = 0; hh < HALVES; ++hh)
-          tma_load_2d(Qs + t * Q_BYTES + hh * QHALF_BYTES, &map_q, q_full, h * D + hh * 64,
-                      row0 + qb * 2 * A2_BM + t * A2_BM);
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int hh = 0; hh < HALVES; ++hh)
+            tma_load_2d(Qs + t * Q_BYTES + hh * QHALF_BYTES, &map_q, q_full, h * D + hh * 64,
+                        row0 + qb * BROWS + t * A2_BM);
+      }
     }
     // The warp looks up the pages of several tiles at a time, lane (i, pg) the page pg of the
     // i-th of them: one gather of the block table per 32 / pages tiles, and per tile little
@@ -271,10 +295,11 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
                                ((uint32_t)(D >> 3) << 17) | ((uint32_t)(A2_BM >> 4) << 24);
       const uint32_t q_addr = smem_u32(Qs + grp * Q_BYTES);
       auto issue_s = [&](int n) {                        // S of tile n into S buffer n & 1
-        const uint32_t k_addr = smem_u32(Ks + (n % A2_STAGES) * KV_BYTES);
+        const uint32_t k_addr =
+            smem_u32(Ks + (n % A2_STAGES) * KV_BYTES + (DIFF ? grp * KHALF_BYTES : 0));
         const uint32_t d_addr = tmem_base + (uint32_t)(grp * 128 + (n & 1) * A2_BN);
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
+        for (int k = 0; k < (DIFF ? 64 : D) / 16; ++k) {
           const uint32_t qo = (uint32_t)((k >> 2) * QHALF_BYTES + (k & 3) * 32);
           const uint32_t ko = (uint32_t)((k >> 2) * KHALF_BYTES + (k & 3) * 32);
           umma_bf16(d_addr, umma_desc_k_sw128(q_addr + qo), umma_desc_k_sw128(k_addr + ko),
@@ -341,10 +366,16 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int rr = wq * 32 + hb * 16 + (lane >> 2) + 8 * e;      // query row of the tile
-        const int ll = qb * 2 * A2_BM + grp * A2_BM + rr;             // index inside the portion
+        const int ll = qb * BROWS + grp * TSHIFT + rr;                // index inside the portion
         validr[e] = ll < qlen;
         prr[e] = pos0 + ll;
         jlr[e] = window > 0 ? max(0, prr[e] - window + 1) : 0;
+      }
+      float row_scale[2] = {scale_log2, scale_log2};     // DIFF: times the row's temperature
+      if constexpr (DIFF) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          row_scale[e] *= bf_query_temperature(prr[e], dd.temp_coef, dd.temp_every);
       }
       uint64_t* my_s_full = s_full + grp * 2;
       uint64_t* my_o_done = o_done + grp * 2;
@@ -359,7 +390,7 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
         tc_fence_after();
         uint32_t v[32];            // v[4c + 2e + i]: row e, key column 8c + 2 q4 + i
         tmem_ld_frag64(my_s + (uint32_t)((n & 1) * A2_BN), v);
-        if (cap_pre > 0.f) {     // s <- (c / scale) tanh(s scale / c): the scale still rides below
+        if (!DIFF && cap_pre > 0.f) {     // s <- (c / scale) tanh(s scale / c): the scale still rides below
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const float t = ex2_approx(__uint_as_float(v[i]) * cap_pre);
@@ -392,7 +423,7 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
           float t = fmaxf(t2[0], t2[1]);
           t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, 1));
           t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, 2));
-          tmax[e] = t * scale_log2;                        // the scale is positive
+          tmax[e] = t * (DIFF ? row_scale[e] : scale_log2);   // the scale is positive
         }
         float factor[2] = {1.f, 1.f};
         bool rescale = false;
@@ -437,7 +468,7 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
           for (int c = 0; c < 8; ++c) {
             float x0, x1;
             fma2f(x0, x1, __uint_as_float(v[4 * c + 2 * e]), __uint_as_float(v[4 * c + 2 * e + 1]),
-                  scale_log2, -m_use);
+                  DIFF ? row_scale[e] : scale_log2, -m_use);
             float e0 = ex2_approx(x0), e1 = ex2_approx(x1);
             if (need_mask[e]) {
               if (8 * c < lo[e] || 8 * c > hi[e]) e0 = 0.f;
@@ -474,7 +505,7 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
       // quarter one half of its columns
       const int half = hb;
       const int r = wq * 32 + lane;
-      const int l = qb * 2 * A2_BM + grp * A2_BM + r;
+      const int l = qb * BROWS + grp * TSHIFT + r;
       const bool valid = l < qlen;
       const uint32_t my_o = tmem_base + ((uint32_t)(wq * 32) << 16) +
                             (uint32_t)(256 + grp * 128 + half * OH);
@@ -482,11 +513,18 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
       bool ok = alive && !*abort &&
                 mbar_wait(my_o_done + ((my_tiles - 1) & 1), (uint32_t)((my_tiles - 1) >> 1) & 1u,
                           abort);
-      ok = group_all(bar_id, ok);
+      // (DIFF without splits: both groups meet, each needs the other's O and sums)
+      if (DIFF && splits == 1) {
+        tc_fence_before();
+        ok = group_all<512>(1, ok);
+      } else {
+        ok = group_all(bar_id, ok);
+      }
       if (ok && splits > 1) {
         // unnormalised, for the merge: O in float, the reference and the sum beside it
         tc_fence_after();
-        const size_t slot = ((size_t)(row0 + l) * nh + h) * splits + split;
+        const size_t slot = (DIFF ? (((size_t)(row0 + l) * nh + h) * 2 + grp)
+                                  : ((size_t)(row0 + l) * nh + h)) * splits + split;
         float* dst = part_o + slot * D + half * OH;
 #pragma unroll 1
         for (int c0 = 0; c0 < OH; c0 += 32) {
@@ -501,6 +539,57 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
         if (valid && half == 0) {
           part_ml[slot * 2] = xr[r];
           part_ml[slot * 2 + 1] = xl[r];
+        }
+      } else if (DIFF) {
+        // this warp's 32 columns of both maps: their difference, its sum of squares shared
+        // with the three other warps of these rows, the norm, the gate
+        const int quarter = grp * 2 + hb;
+        float diff[32];
+        float ss = 0.f;
+        if (ok) {
+          tc_fence_after();
+          const uint32_t my_a = tmem_base + ((uint32_t)(wq * 32) << 16) +
+                                (uint32_t)(256 + quarter * 32);
+          const float inv_a = 1.f / xm[r], inv_b = dd.lambda / xm[128 + r];
+          uint32_t w[32];
+          tmem_ld32(my_a, w);
+#pragma unroll
+          for (int c = 0; c < 32; ++c) diff[c] = __uint_as_float(w[c]) * inv_a;
+          tmem_ld32(my_a + 128, w);
+#pragma unroll
+          for (int c = 0; c < 32; ++c) {
+            diff[c] -= __uint_as_float(w[c]) * inv_b;
+            ss += diff[c] * diff[c];
+          }
+          xss[quarter * 128 + r] = ss;
+        }
+        group_all<512>(1, ok);
+        if (ok && valid) {
+          const float f = rsqrtf((((xss[r] + xss[128 + r]) + xss[256 + r]) + xss[384 + r]) *
+                                     (1.f / (float)D) + dd.eps) * dd.out_factor;
+          const size_t col = (size_t)h * D + quarter * 32;
+          const __nv_bfloat16* gate =
+              dd.gate ? (const __nv_bfloat16*)dd.gate + (size_t)(row0 + l) * dd.gate_stride + col
+                      : nullptr;
+          __nv_bfloat16* dst = out + (size_t)(row0 + l) * out_stride + col;
+#pragma unroll
+          for (int c = 0; c < 32; c += 8) {
+            uint4 g4 = make_uint4(0u, 0u, 0u, 0u), o4;
+            if (gate) g4 = *reinterpret_cast<const uint4*>(gate + c);
+            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
+            __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              float a = diff[c + 2 * j] * f, b = diff[c + 2 * j + 1] * f;
+              if (gate) {
+                const float2 gv = __bfloat1622float2(g2[j]);
+                a *= bf_sigmoid_fast(gv.x);
+                b *= bf_sigmoid_fast(gv.y);
+              }
+              o2[j] = __floats2bfloat162_rn(a, b);
+            }
+            *reinterpret_cast<uint4*>(dst + c) = o4;
+          }
         }
       } else if (ok) {
         tc_fence_after();
@@ -527,9 +616,10 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
       tc_fence_before();
     } else if (splits > 1 && (grp == 0 || active_b) && ((warp >> 2) & 1) == 0) {
       // no key tile of this share for the group's rows: a partial that the merge passes over
-      const int l = qb * 2 * A2_BM + grp * A2_BM + (warp & 3) * 32 + lane;
+      const int l = qb * BROWS + grp * TSHIFT + (warp & 3) * 32 + lane;
       if (l < qlen) {
-        const size_t slot = ((size_t)(row0 + l) * nh + h) * splits + split;
+        const size_t slot = (DIFF ? (((size_t)(row0 + l) * nh + h) * 2 + grp)
+                                  : ((size_t)(row0 + l) * nh + h)) * splits + split;
         part_ml[slot * 2] = -INFINITY;
         part_ml[slot * 2 + 1] = 0.f;
       }
@@ -627,7 +717,7 @@ BF_EXPORT int bf_prefill_attention_umma2_capped(
   if (e) return e;
   // two Q tiles, the stages of K and V, the row sums, barriers
   const size_t smem = 1024 + (size_t)2 * 32768 + (size_t)2 * A2_STAGES * 16384 + 2048 + 256;
-  auto kern = prefill_attention_umma2_kernel;
+  auto kern = prefill_attention_umma2_kernel<false>;
   static bool configured_on[BF_MAX_DEVICES];
   bool& configured = configured_on[bf_current_device()];
   if (!configured) {
@@ -641,7 +731,8 @@ BF_EXPORT int bf_prefill_attention_umma2_capped(
   kern<<<grid, A2_THREADS, smem, stream>>>(mq, mk, mv, mkr, mvr, items, block_tables, table_stride,
                                            (__nv_bfloat16*)out, nh, nkv, page_size, num_pages,
                                            window, scale * log2e, splits, part_o, part_ml, err,
-                                           cap_pre, cap_post, out_stride, out_scale);
+                                           cap_pre, cap_post, out_stride, out_scale,
+                                           BfDiffArgs());
   if (splits > 1) {
     int st = bf_launch_status();
     if (st) return st;
@@ -662,4 +753,64 @@ BF_EXPORT int bf_prefill_attention_umma2(const void* q, const void* k_cache, con
                                            total_rows, block_tables, table_stride, out, nh, nkv,
                                            d, page_size, num_pages, window, scale, splits, part_o,
                                            part_ml, err, 0.f, (long long)nh * A2_D, 1.f, stream);
+}
+
+// Differential attention of prompt portions: heads of two maps with 64 key columns each (a cached
+// key row holds both, 128) over values of 128.  q: rows `q_stride` elements apart, head h's maps
+// at columns h 128 and h 128 + 64.  The other arguments as above (nh query heads, part_o
+// [total_rows, nh, 2, splits, 128], part_ml likewise); lambda, the norm's eps, the output's
+// factor, the gate (rows `gate_stride` apart, or null) and the query temperature: attention_diff.cuh.
+BF_EXPORT int bf_diff_attention_prefill_umma(
+    const void* q, long long q_stride, const void* k_cache, const void* v_cache, const int* items,
+    int n_items, int max_rows, int total_rows, const int* block_tables, int table_stride,
+    void* out, int nh, int nkv, int page_size, int num_pages, float scale, int splits,
+    float* part_o, float* part_ml, int* err, long long out_stride, const void* gate,
+    long long gate_stride, float lambda, float eps, float out_factor, float temp_coef,
+    int temp_every, cudaStream_t stream) {
+  if (n_items <= 0 || max_rows <= 0) return 0;
+  if (splits < 1 || (splits > 1 && (!part_o || !part_ml))) return (int)cudaErrorInvalidValue;
+  if (nkv <= 0 || nh % nkv || page_size < 8 || page_size > A2_BN || A2_BN % page_size ||
+      ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) ||
+      ((uintptr_t)out & 15) || !(scale > 0.f) || out_stride < (long long)nh * A2_D ||
+      (out_stride & 7) || (q_stride & 7) || q_stride < (long long)nh * A2_D ||
+      ((uintptr_t)gate & 15) || (gate_stride & 7) || temp_every < 1 || temp_coef < 0.f)
+    return (int)cudaErrorInvalidValue;
+  CUtensorMap mq, mk, mv, mkr, mvr;
+  int e = bf_make_tensor_map_bf16_2d(&mq, q, total_rows, (long long)nh * A2_D, q_stride, A2_BM, 64);
+  if (e) return e;
+  const long long cache_rows = (long long)num_pages * nkv * page_size;
+  e = bf_make_tensor_map_bf16_2d(&mk, k_cache, cache_rows, A2_D, A2_D, page_size, 64);
+  if (e) return e;
+  e = bf_make_tensor_map_bf16_2d(&mv, v_cache, cache_rows, A2_D, A2_D, page_size, 64);
+  if (e) return e;
+  e = bf_make_tensor_map_pages_bf16(&mkr, k_cache, num_pages, nkv, page_size, A2_D,
+                                    A2_BN / page_size);
+  if (e) return e;
+  e = bf_make_tensor_map_pages_bf16(&mvr, v_cache, num_pages, nkv, page_size, A2_D,
+                                    A2_BN / page_size);
+  if (e) return e;
+  const size_t smem = 1024 + (size_t)2 * 32768 + (size_t)2 * A2_STAGES * 16384 + 4096 + 256;
+  auto kern = prefill_attention_umma2_kernel<true>;
+  static bool configured_on[BF_MAX_DEVICES];
+  bool& configured = configured_on[bf_current_device()];
+  if (!configured) {
+    cudaError_t ce = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                          (int)smem);
+    if (ce != cudaSuccess) return (int)ce;
+    configured = true;
+  }
+  dim3 grid(nh, n_items * splits, (max_rows + A2_BM - 1) / A2_BM);
+  if (grid.y > 65535u || grid.z > 65535u) return (int)cudaErrorInvalidValue;
+  const BfDiffArgs dd = {gate, gate_stride, lambda, eps, out_factor, temp_coef, temp_every};
+  kern<<<grid, A2_THREADS, smem, stream>>>(mq, mk, mv, mkr, mvr, items, block_tables, table_stride,
+                                           (__nv_bfloat16*)out, nh, nkv, page_size, num_pages, 0,
+                                           scale * 1.4426950408889634f, splits, part_o, part_ml,
+                                           err, 0.f, 0.f, out_stride, 1.f, dd);
+  if (splits > 1) {
+    int st = bf_launch_status();
+    if (st) return st;
+    return bf_diff_attention_merge_items(part_o, part_ml, items, n_items, max_rows, out, nh, A2_D,
+                                         splits, out_stride, dd, stream);
+  }
+  return bf_launch_status();
 }

@@ -24,10 +24,14 @@ BF_EXPORT void bf_set_pdl(int on) { g_pdl = on ? 1 : 0; }
 // ------------------------------------------------------------------ embedding
 // out[t, :] = table[ids[t], :] * scale   (cuda/kernels/bf16_kernels.cu:711-729,
 // which does not check the id; here a bad id sets an error bit and yields zeros).
+// With `freqs` (double, one per pair of columns) a sinusoidal vector of the token's position is
+// added: column 2i gets sin(p f_i), column 2i + 1 cos(p f_i).  The angle is formed and reduced
+// to one turn in double, so that far positions lose nothing; sine and cosine are float.
 template <typename W>
 __global__ void embed_gather_kernel(const W* __restrict__ table, const int* __restrict__ ids,
                                     float* __restrict__ out, int H, int vocab, float scale,
-                                    int* __restrict__ err) {
+                                    int* __restrict__ err, const int* __restrict__ positions,
+                                    const double* __restrict__ freqs) {
   bf_pdl_trigger();
   bf_pdl_wait();
   const int t = blockIdx.x;
@@ -39,19 +43,32 @@ __global__ void embed_gather_kernel(const W* __restrict__ table, const int* __re
     return;
   }
   const W* row = table + (size_t)id * H;
+  if (freqs) {
+    const double p = (double)positions[t];
+    for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
+      const double turns = p * freqs[i] * 0.15915494309189535;      // over 2 pi
+      float sn, cs;
+      sincospif(2.f * (float)(turns - floor(turns)), &sn, &cs);
+      o[2 * i] = bf_ld(row + 2 * i) * scale + sn;
+      if (2 * i + 1 < H) o[2 * i + 1] = bf_ld(row + 2 * i + 1) * scale + cs;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = bf_ld(row + i) * scale;
 }
 
 BF_EXPORT int bf_embed_gather(const void* table, int table_dtype, const int* ids, float* out,
                               int T, int H, int vocab, float scale, int* err,
-                              cudaStream_t stream) {
+                              const int* positions, const double* freqs, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (!positions) freqs = nullptr;
   const int threads = H >= 1024 ? 256 : 128;
   if (table_dtype == BF_DTYPE_F32)
     return bf_launch_pdl(embed_gather_kernel<float>, dim3(T), dim3(threads), 0, stream,
-                         (const float*)table, ids, out, H, vocab, scale, err);
+                         (const float*)table, ids, out, H, vocab, scale, err, positions, freqs);
   return bf_launch_pdl(embed_gather_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream,
-                       (const __nv_bfloat16*)table, ids, out, H, vocab, scale, err);
+                       (const __nv_bfloat16*)table, ids, out, H, vocab, scale, err, positions,
+                       freqs);
 }
 
 // -------------------------------------------------------- add + RMSNorm (fused)
@@ -219,16 +236,28 @@ BF_EXPORT int bf_residual_add(float* resid, const void* delta, long long n, int 
 // here they are the two halves of one fused projection's output row).
 // ACT 1: the tanh form of gelu in silu's place,
 //   gelu(g) = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
+// ACT 2: clamped, with three constants: g = min(gate, limit), u = clamp(up, -limit, limit),
+//   g sigmoid(slope g) (u + up_offset).
 #define BF_ACT_SILU 0
 #define BF_ACT_GELU_TANH 1
+#define BF_ACT_CLAMPED 2
+struct BfGateConst {
+  float limit, slope, up_offset;
+};
 template <int ACT>
-__device__ __forceinline__ float bf_gate_act(float g) {
+__device__ __forceinline__ float bf_gate_mul(float g, float u, const BfGateConst& k) {
+  if (ACT == BF_ACT_CLAMPED) {
+    g = fminf(g, k.limit);
+    u = fminf(fmaxf(u, -k.limit), k.limit) + k.up_offset;
+    return g / (1.f + expf(-k.slope * g)) * u;
+  }
   if (ACT == BF_ACT_GELU_TANH)
-    return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-  return g / (1.f + expf(-g));
+    return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  return g / (1.f + expf(-g)) * u;
 }
 template <typename A, int ACT>
-__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, int T, int I) {
+__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, int T, int I,
+                                BfGateConst gk) {
   const size_t n = (size_t)T * I;
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
@@ -236,7 +265,7 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, i
     const size_t t = i / I, c = i - t * I;
     const float g = bf_ld(gu + t * 2 * I + c);
     const float u = bf_ld(gu + t * 2 * I + I + c);
-    bf_st(out + i, bf_gate_act<ACT>(g) * u);
+    bf_st(out + i, bf_gate_mul<ACT>(g, u, gk));
   }
 }
 
@@ -246,12 +275,17 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, i
 __device__ __forceinline__ float bf_silu_fast(float g) { return __fdividef(g, 1.f + __expf(-g)); }
 // ... and gelu's tanh form the same way: 0.5 g (1 + tanh(z)) = g / (1 + exp(-2 z))
 template <int ACT>
-__device__ __forceinline__ float bf_gate_act_fast(float g) {
+__device__ __forceinline__ float bf_gate_mul_fast(float g, float u, const BfGateConst& k) {
+  if (ACT == BF_ACT_CLAMPED) {
+    g = fminf(g, k.limit);
+    u = fminf(fmaxf(u, -k.limit), k.limit) + k.up_offset;
+    return __fdividef(g, 1.f + __expf(-k.slope * g)) * u;
+  }
   if (ACT == BF_ACT_GELU_TANH) {
     const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-    return __fdividef(g, 1.f + __expf(-2.f * z));
+    return __fdividef(g, 1.f + __expf(-2.f * z)) * u;
   }
-  return bf_silu_fast(g);
+  return bf_silu_fast(g) * u;
 }
 
 // The same when the rows of gu still lack a factor (see BfRowScale).  I is at least 256, so
@@ -305,7 +339,8 @@ __global__ void silu_mul_bf16_scaled_kernel(const __nv_bfloat16* __restrict__ gu
 // bf16, I a multiple of 8: eight elements per thread with 16-byte loads and stores.
 template <int ACT>
 __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
-                                         __nv_bfloat16* __restrict__ out, int T, int I) {
+                                         __nv_bfloat16* __restrict__ out, int T, int I,
+                                         BfGateConst gk) {
   BF_TRACE_POINT(10 * BF_TR_SILU);
   bf_pdl_trigger();
   bf_pdl_wait();
@@ -335,7 +370,8 @@ __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
-        o2[j] = __floats2bfloat162_rn(bf_gate_act_fast<ACT>(g.x) * u.x, bf_gate_act_fast<ACT>(g.y) * u.y);
+        o2[j] = __floats2bfloat162_rn(bf_gate_mul_fast<ACT>(g.x, u.x, gk),
+                                      bf_gate_mul_fast<ACT>(g.y, u.y, gk));
       }
       *reinterpret_cast<uint4*>(out + (k ? t2 * I + c2 : t * I + c)) = o4;
     }
@@ -361,7 +397,7 @@ BF_EXPORT int bf_silu_mul_scaled(const void* gu, void* out, int T, int I,
 
 template <int ACT>
 static int gated_act_mul_launch(const void* gu, void* out, int T, int I, int act_dtype,
-                                cudaStream_t stream) {
+                                cudaStream_t stream, BfGateConst gk = BfGateConst()) {
   if (T <= 0) return 0;
   const int threads = 256;
   if (act_dtype == BF_DTYPE_BF16 && I % 8 == 0 && ((uintptr_t)gu & 15) == 0 &&
@@ -369,16 +405,16 @@ static int gated_act_mul_launch(const void* gu, void* out, int T, int I, int act
     long long blocks = ((long long)T * (I / 8) + threads - 1) / threads;
     if (blocks > 148 * 16) blocks = 148 * 16;
     return bf_launch_pdl(silu_mul_bf16_vec_kernel<ACT>, dim3((int)blocks), dim3(threads), 0,
-                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I);
+                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk);
   }
   long long blocks = ((long long)T * I + threads - 1) / threads;
   if (blocks > 148 * 32) blocks = 148 * 32;
   if (act_dtype == BF_DTYPE_F32)
     silu_mul_kernel<float, ACT><<<(int)blocks, threads, 0, stream>>>((const float*)gu,
-                                                                    (float*)out, T, I);
+                                                                    (float*)out, T, I, gk);
   else
     silu_mul_kernel<__nv_bfloat16, ACT><<<(int)blocks, threads, 0, stream>>>(
-        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I);
+        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk);
   return bf_launch_status();
 }
 
@@ -387,9 +423,13 @@ BF_EXPORT int bf_silu_mul(const void* gu, void* out, int T, int I, int act_dtype
   return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream);
 }
 
-// out[t, c] = act(gu[t, c]) * gu[t, I + c] with act 0: silu, 1: gelu's tanh form.
+// out[t, c] = act(gu[t, c]) * gu[t, I + c] with act 0: silu, 1: gelu's tanh form; 2: the clamped
+// form with its three constants (see BF_ACT_CLAMPED).
 BF_EXPORT int bf_gated_act_mul(const void* gu, void* out, int T, int I, int act, int act_dtype,
-                               cudaStream_t stream) {
+                               float limit, float slope, float up_offset, cudaStream_t stream) {
+  if (act == BF_ACT_CLAMPED)
+    return gated_act_mul_launch<BF_ACT_CLAMPED>(gu, out, T, I, act_dtype, stream,
+                                                BfGateConst{limit, slope, up_offset});
   if (act == BF_ACT_SILU) return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream);
   if (act == BF_ACT_GELU_TANH)
     return gated_act_mul_launch<BF_ACT_GELU_TANH>(gu, out, T, I, act_dtype, stream);

@@ -16,6 +16,10 @@
 // are added up in a column of their own behind the experts' (and the shared gate's), and
 // bf_moe_identity_add adds input times that column to the mixture's output.
 //
+// Two variations of that way: the scores may be the sigmoids of the outputs instead (`mode` 2),
+// a group may count by the sum of its `group_top` largest choice scores, and the chosen scores
+// may stay as they are (`normalize` 0: no division by their sum).
+//
 // moe_act: for experts whose gate and up projections are stacked into one product
 // `gu [T, 2F]` (gate rows of all experts, then up rows; F = E ff + ff_shared), the
 // activations of every expert scaled by the token's weight for that expert,
@@ -39,7 +43,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     int E, int top, int shared_gate, int tokens_per_block, float* __restrict__ route_w,
     int* __restrict__ top_ids, float* __restrict__ top_w, int mode,
     const float* __restrict__ correction, int n_groups, int keep, int identity,
-    float route_scale, float weight_eps) {
+    float route_scale, float weight_eps, int group_top, int normalize) {
   extern __shared__ __align__(16) float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * tokens_per_block;
@@ -122,18 +126,19 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
   for (int e = lane; e < rw_cols; e += 32) rw[e] = 0.f;
   if (shared_gate && lane == 0) rw[E] = 1.f / (1.f + expf(-z[R]));
   __syncwarp();
-  if (mode == 1) {
+  if (mode != 0) {
     float* ch = chs + (size_t)warp * rows;
     // this warp's slice of the partial sums' place, which nobody reads any more
     float* gsc = part + (size_t)warp * MR_TOKENS * rows;   // [n_groups] scores, [n_groups] kept
-    float zmax = -FLT_MAX;
-    for (int e = lane; e < R; e += 32) zmax = fmaxf(zmax, z[e]);
-    zmax = warp_max(zmax);
-    float den = 0.f;
-    for (int e = lane; e < R; e += 32) den += expf(z[e] - zmax);
-    den = warp_sum(den);
+    float zmax = -FLT_MAX, den = 0.f;
+    if (mode == 1) {
+      for (int e = lane; e < R; e += 32) zmax = fmaxf(zmax, z[e]);
+      zmax = warp_max(zmax);
+      for (int e = lane; e < R; e += 32) den += expf(z[e] - zmax);
+      den = warp_sum(den);
+    }
     for (int e = lane; e < R; e += 32) {
-      const float sc = expf(z[e] - zmax) / den;
+      const float sc = mode == 1 ? expf(z[e] - zmax) / den : 1.f / (1.f + expf(-z[e]));
       z[e] = sc;
       ch[e] = sc + (correction ? correction[e] : 0.f);
     }
@@ -141,9 +146,25 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     if (n_groups > 1) {
       const int per = R / n_groups;
       for (int g = lane; g < n_groups; g += 32) {
-        float best = -FLT_MAX;
-        for (int i = 0; i < per; ++i) best = fmaxf(best, ch[g * per + i]);
-        gsc[g] = best;
+        // the sum of the group's `group_top` largest, one after the other: a walk finds the
+        // largest value below the last one, or equal to it at a later place
+        float sum_g = 0.f, last = FLT_MAX;
+        int last_i = -1;
+        for (int k = 0; k < group_top && k < per; ++k) {
+          float best = -FLT_MAX;
+          int at = per;
+          for (int i = 0; i < per; ++i) {
+            const float c = ch[g * per + i];
+            if ((c < last || (c == last && i > last_i)) && (at == per || c > best)) {
+              best = c;
+              at = i;
+            }
+          }
+          sum_g += best;
+          last = best;
+          last_i = at;
+        }
+        gsc[g] = sum_g;
         gsc[n_groups + g] = 0.f;
       }
       __syncwarp();
@@ -193,7 +214,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
       }
       __syncwarp();
     }
-    const float f = route_scale / (sum + weight_eps);
+    const float f = normalize ? route_scale / (sum + weight_eps) : route_scale;
     if (lane == 0) {
       for (int k = 0; k < top; ++k) {
         const float pw = top_w[(size_t)t * top + k] * f;
@@ -242,8 +263,10 @@ BF_EXPORT int bf_moe_route(const void* h, long long stride, const float* w, int 
                            int E, int top, int shared_gate, float* route_w, int* top_ids,
                            float* top_w, int act_dtype, int mode, const float* correction,
                            int n_groups, int keep, int identity, float route_scale,
-                           float weight_eps, cudaStream_t stream) {
+                           float weight_eps, int group_top, int normalize,
+                           cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (group_top < 1) return (int)cudaErrorInvalidValue;
   if (mode == 0) { identity = 0; n_groups = 1; correction = nullptr; }
   if (n_groups < 1) n_groups = 1;
   if (top < 1 || top > E + identity || identity < 0 || (E + identity) % n_groups ||
@@ -263,7 +286,7 @@ BF_EXPORT int bf_moe_route(const void* h, long long stride, const float* w, int 
     k<<<blocks, MR_WARPS * 32, smem, stream>>>((const float*)h, stride, w, T, width, E, top,
                                                shared_gate, tpb, route_w, top_ids, top_w, mode,
                                                correction, n_groups, keep, identity, route_scale,
-                                               weight_eps);
+                                               weight_eps, group_top, normalize);
   } else {
     auto k = moe_route_kernel<__nv_bfloat16>;
     if (smem > 48 * 1024)
@@ -271,7 +294,7 @@ BF_EXPORT int bf_moe_route(const void* h, long long stride, const float* w, int 
     k<<<blocks, MR_WARPS * 32, smem, stream>>>((const __nv_bfloat16*)h, stride, w, T, width, E,
                                                top, shared_gate, tpb, route_w, top_ids, top_w,
                                                mode, correction, n_groups, keep, identity,
-                                               route_scale, weight_eps);
+                                               route_scale, weight_eps, group_top, normalize);
   }
   return bf_launch_status();
 }

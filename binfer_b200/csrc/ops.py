@@ -107,13 +107,22 @@ def _want(t: torch.Tensor, dtype: torch.dtype, name: str) -> None:
 
 # ------------------------------------------------------------------ elementwise
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float,
-                 err: torch.Tensor) -> None:
-    """out[t] = table[ids[t]] * scale; out is the float residual stream [T, H]."""
+                 err: torch.Tensor, positions: Optional[torch.Tensor] = None,
+                 freqs: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[ids[t]] * scale; out is the float residual stream [T, H].  With ``freqs``
+    (float64, one per pair of columns) sin(positions[t] freqs[i]) is added to column 2i and the
+    cosine to column 2i + 1."""
     _want(ids, torch.int32, "ids"); _want(out, torch.float32, "out")
     T, H = out.shape
+    if (freqs is None) != (positions is None):
+        raise KernelError("embed_gather: positions and freqs go together")
+    if freqs is not None:
+        _want(positions, torch.int32, "positions"); _want(freqs, torch.float64, "freqs")
+        if freqs.numel() != (H + 1) // 2:
+            raise KernelError("embed_gather: freqs must have one number per pair of columns")
     _run("embed_gather", lib().bf_embed_gather, _ptr(table), _c_int(_dtype_code(table)), _ptr(ids), _ptr(out),
                                  _c_int(T), _c_int(H), _c_int(table.shape[0]), _c_float(scale),
-                                 _ptr(err), _stream())
+                                 _ptr(err), _ptr(positions), _ptr(freqs), _stream())
 
 
 def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor,
@@ -182,19 +191,22 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor,
                              _c_int(_dtype_code(out)), _stream())
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
 
 
-def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str) -> None:
+def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str,
+                  limit: float = 0.0, slope: float = 1.0, up_offset: float = 0.0) -> None:
     """out[t, c] = act(gate_up[t, c]) * gate_up[t, I + c]; ``activation`` one of
-    ``GATE_ACTIVATIONS``."""
+    ``GATE_ACTIVATIONS``.  "clamped": with g = min(gate, limit) and u = clamp(up, -limit, limit)
+    the result is g sigmoid(slope g) (u + up_offset)."""
     T, I = out.shape
     if activation not in GATE_ACTIVATIONS:
         raise KernelError(f"gated_act_mul: unknown activation {activation!r}")
     if gate_up.shape != (T, 2 * I) or not gate_up.is_contiguous() or gate_up.dtype != out.dtype:
         raise KernelError("gated_act_mul: gate_up must be contiguous [T, 2*I] of the output's dtype")
     _run("gated_act_mul", lib().bf_gated_act_mul, _ptr(gate_up), _ptr(out), _c_int(T), _c_int(I),
-         _c_int(GATE_ACTIVATIONS[activation]), _c_int(_dtype_code(out)), _stream())
+         _c_int(GATE_ACTIVATIONS[activation]), _c_int(_dtype_code(out)), _c_float(limit),
+         _c_float(slope), _c_float(up_offset), _stream())
 
 
 def copy_ids(dst: torch.Tensor, src: torch.Tensor, pairs: torch.Tensor, n: int) -> None:
@@ -935,11 +947,15 @@ def stream_inject(resid: torch.Tensor, delta: Optional[torch.Tensor],
 
 
 # ---------------------------------------------------------------- mixture of experts
+MOE_SCORINGS = {"softmax_top": 0, "softmax_all": 1, "sigmoid": 2}
+
+
 def moe_route(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, shared_gate: bool,
               route_w: torch.Tensor, top_ids: torch.Tensor, top_w: torch.Tensor,
               scoring: str = "softmax_top", correction: Optional[torch.Tensor] = None,
               groups: int = 1, groups_keep: int = 1, identity: int = 0,
-              route_scale: float = 1.0, weight_eps: float = 0.0) -> None:
+              route_scale: float = 1.0, weight_eps: float = 0.0, group_top: int = 1,
+              normalize: bool = True) -> None:
     """Router of a mixture of experts: ``w`` float32 ``[experts + identity (+1), width]`` (the
     last row the shared expert's gate when ``shared_gate``), ``h [T, width]``.  ``route_w``
     float32 ``[T, experts (+1) (+1)]`` gets every expert's weight for the token (zero: not
@@ -952,14 +968,18 @@ def moe_route(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, shared_g
     outputs, ``correction`` (float32, one number per output) is added for the choice only,
     with ``groups`` > 1 only the outputs of the ``groups_keep`` groups with the largest best
     choice score can be chosen, and the weights are the chosen scores over their sum (plus
-    ``weight_eps``) times ``route_scale``."""
+    ``weight_eps``) times ``route_scale``.  "sigmoid": the same with the sigmoids of the outputs
+    as scores.  ``group_top``: a group counts by the sum of its that many largest choice scores;
+    ``normalize`` False: the chosen scores are not divided by their sum."""
     T, width = h.shape
-    if scoring not in ("softmax_top", "softmax_all"):
+    if scoring not in MOE_SCORINGS:
         raise KernelError(f"moe_route: unknown scoring {scoring!r}")
-    mode = 1 if scoring == "softmax_all" else 0
-    if mode == 0 and (identity or groups > 1 or correction is not None):
-        raise KernelError("moe_route: corrections, groups and identity outputs go with the "
-                          "softmax over all outputs")
+    mode = MOE_SCORINGS[scoring]
+    if mode == 0 and (identity or groups > 1 or correction is not None or not normalize):
+        raise KernelError("moe_route: corrections, groups, identity outputs and scores that are "
+                          "not normalized go with scores over all outputs")
+    if group_top < 1:
+        raise KernelError("moe_route: group_top must be positive")
     rows = experts + identity + (1 if shared_gate else 0)
     cols = experts + (1 if shared_gate else 0) + (1 if identity else 0)
     _want(w, torch.float32, "w"); _want(route_w, torch.float32, "route_w")
@@ -980,7 +1000,8 @@ def moe_route(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, shared_g
          _c_int(width), _c_int(experts), _c_int(top), _c_int(1 if shared_gate else 0),
          _ptr(route_w), _ptr(top_ids), _ptr(top_w), _c_int(_dtype_code(h)), _c_int(mode),
          _ptr(correction), _c_int(groups), _c_int(groups_keep), _c_int(identity),
-         _c_float(route_scale), _c_float(weight_eps), _stream())
+         _c_float(route_scale), _c_float(weight_eps), _c_int(group_top),
+         _c_int(1 if normalize else 0), _stream())
 
 
 def moe_act(gu: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor, experts: int,
@@ -1056,9 +1077,12 @@ def moe_sparse(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
 
 # ----------------------------------------------------- norm on a sublayer's output
 def rmsnorm_add(resid: torch.Tensor, y: torch.Tensor, weight: torch.Tensor,
-                reading: Optional[torch.Tensor], eps: float) -> None:
+                reading: Optional[torch.Tensor], eps: float,
+                next_weight: Optional[torch.Tensor] = None, next_eps: float = 0.0) -> None:
     """``resid += y * rsqrt(mean(y^2) + eps) * weight`` row by row (``resid`` float32
-    ``[T, H]``), and, if ``reading`` is given, the new rows in its type."""
+    ``[T, H]``), and, if ``reading`` is given, the new rows in its type.  With ``next_weight``
+    (float32 ``[H]``) ``reading`` gets the new rows through the norm that reads them next
+    instead, ``resid * rsqrt(mean(resid^2) + next_eps) * next_weight``."""
     _want(resid, torch.float32, "resid"); _want(weight, torch.float32, "weight")
     T, H = resid.shape
     if y.shape != resid.shape or not y.is_contiguous():
@@ -1066,8 +1090,13 @@ def rmsnorm_add(resid: torch.Tensor, y: torch.Tensor, weight: torch.Tensor,
     if reading is not None and (reading.dtype != y.dtype or reading.shape != resid.shape
                                 or not reading.is_contiguous()):
         raise KernelError("rmsnorm_add: the reading must be contiguous, of y's type and shape")
+    if next_weight is not None:
+        _want(next_weight, torch.float32, "next_weight")
+        if reading is None or next_weight.numel() != H:
+            raise KernelError("rmsnorm_add: a next norm needs an output and a weight of the width")
     _run("rmsnorm_add", lib().bf_rmsnorm_add, _ptr(resid), _ptr(y), _ptr(weight), _ptr(reading),
-         _c_int(T), _c_int(H), _c_float(eps), _c_int(_dtype_code(y)), _stream())
+         _c_int(T), _c_int(H), _c_float(eps), _c_int(_dtype_code(y)), _ptr(next_weight),
+         _c_float(next_eps), _stream())
 
 
 def stream_to_bf16(x: torch.Tensor, out: torch.Tensor) -> None:
@@ -1333,6 +1362,184 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tensor
 
 
 # ------------------------------------------------------------- matrix products
+# ------------------------------------------------------------- differential attention
+def kv_store(proj: torch.Tensor, k_off: int, v_off: int, slots: torch.Tensor,
+             k_cache: torch.Tensor, v_cache: torch.Tensor, err: torch.Tensor) -> None:
+    """Key heads (columns ``k_off ..`` of ``proj``) and value heads (``v_off ..``) of every token
+    into its place ``slots[t]`` of the pages ``k_cache [pages, heads, page_size, dk]`` and
+    ``v_cache [..., dv]``."""
+    T = proj.shape[0]
+    nkv, ps, dk = k_cache.shape[1:]
+    dv = v_cache.shape[3]
+    _want(slots, torch.int32, "slots")
+    if (proj.stride(1) != 1 or proj.dtype != k_cache.dtype or v_cache.dtype != k_cache.dtype
+            or not k_cache.is_contiguous() or not v_cache.is_contiguous()
+            or tuple(v_cache.shape[:3]) != tuple(k_cache.shape[:3]) or slots.numel() < T
+            or max(k_off + nkv * dk, v_off + nkv * dv) > proj.shape[1]):
+        raise KernelError("kv_store: rows of proj must hold the key and value heads of the pages")
+    _run("kv_store", lib().bf_kv_store, _ptr(proj), _c_ll(proj.stride(0)), _c_int(k_off),
+         _c_int(v_off), _ptr(slots), _ptr(k_cache), _ptr(v_cache), _c_int(T), _c_int(nkv),
+         _c_int(dk), _c_int(dv), _c_int(ps), _c_ll(k_cache.shape[0] * ps),
+         _c_int(_dtype_code(proj)), _ptr(err), _stream())
+
+
+class DiffCombine:
+    """What the differential attention kernels do with a head's two maps, besides attending:
+    ``o = a1 - lam a2``, ``o <- o / sqrt(mean(o^2) + eps) * out_factor``, times the sigmoid of
+    ``gate`` (rows of ``heads * dv`` numbers of the activation type, which may be a column block;
+    None: no gate).  The query at position p counts ``1 + temp_coef ln(floor((p + 1) /
+    temp_every) + 1)`` times (``temp_coef`` 0: once)."""
+    __slots__ = ("lam", "eps", "out_factor", "gate", "temp_coef", "temp_every")
+
+    def __init__(self, lam: float, eps: float, out_factor: float,
+                 gate: Optional[torch.Tensor] = None, temp_coef: float = 0.0,
+                 temp_every: int = 1):
+        self.lam, self.eps, self.out_factor, self.gate = lam, eps, out_factor, gate
+        self.temp_coef, self.temp_every = temp_coef, int(temp_every)
+
+    def args(self, q: torch.Tensor, out: torch.Tensor):
+        g = self.gate
+        if g is not None and (g.dtype != q.dtype or g.stride(1) != 1 or g.shape != out.shape):
+            raise KernelError("differential attention: the gate must have the output's shape and "
+                              "type, its rows contiguous")
+        return (_c_ll(out.stride(0)), _ptr(g), _c_ll(g.stride(0) if g is not None else 0),
+                _c_float(self.lam), _c_float(self.eps), _c_float(self.out_factor),
+                _c_float(self.temp_coef), _c_int(self.temp_every))
+
+
+def _diff_check(q, k_cache, v_cache, out, nh, dc):
+    nkv, d2 = k_cache.shape[1], k_cache.shape[3]
+    dv = v_cache.shape[3]
+    if (nh % nkv or d2 % 2 or q.stride(1) != 1 or out.stride(1) != 1 or q.shape[1] != nh * d2
+            or out.shape[1] != nh * dv or q.dtype != k_cache.dtype or out.dtype != q.dtype
+            or not k_cache.is_contiguous() or not v_cache.is_contiguous() or dc.temp_every < 1):
+        raise KernelError("differential attention: q [T, heads * 2 d], key pages of 2 d, value "
+                          "pages of dv, out [T, heads * dv], all of one type")
+    return nkv, d2 // 2, dv
+
+
+DIFF_MAX_DIM = 512
+
+
+def diff_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                           seq_of_token: torch.Tensor, positions: torch.Tensor,
+                           block_tables: torch.Tensor, out: torch.Tensor, nh: int, scale: float,
+                           dc: DiffCombine, err: torch.Tensor) -> None:
+    """Differential attention of every token row over its request's pages, any sizes (float32,
+    and bfloat16 where the tensor-core kernels do not apply).  ``q [T, nh * 2 d]`` holds a
+    head's two query vectors side by side, ``k_cache [pages, nkv, page_size, 2 d]`` likewise,
+    ``v_cache [pages, nkv, page_size, dv]``; ``out [T, nh * dv]``; q and out may be column
+    blocks of wider buffers."""
+    nkv, d, dv = _diff_check(q, k_cache, v_cache, out, nh, dc)
+    if d > DIFF_MAX_DIM or dv > DIFF_MAX_DIM:
+        raise KernelError(f"differential attention: sizes {d}, {dv} are not supported (at most "
+                          f"{DIFF_MAX_DIM})")
+    o_stride, *rest = dc.args(q, out)
+    _run("diff_attention_generic", lib().bf_diff_attention_generic, _ptr(q), _c_ll(q.stride(0)),
+         _ptr(k_cache), _ptr(v_cache), _ptr(seq_of_token), _ptr(positions), _ptr(block_tables),
+         _c_int(block_tables.stride(0)), _ptr(out), o_stride, _c_int(q.shape[0]), _c_int(nh),
+         _c_int(nkv), _c_int(d), _c_int(dv), _c_int(k_cache.shape[2]), _c_int(k_cache.shape[0]),
+         _c_float(scale), _c_int(_dtype_code(q)), _ptr(err), *rest, _stream())
+
+
+def diff_attention_takes(dtype: torch.dtype, d: int, dv: int, scale: float,
+                         temp_coef: float = 0.0) -> bool:
+    """Whether the tensor-core kernels of the differential attention take these sizes."""
+    return (dtype == torch.bfloat16 and d % 16 == 0 and dv % 16 == 0 and 0 < d <= 128
+            and 0 < dv <= 128 and scale > 0 and temp_coef >= 0)
+
+
+def diff_attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                           items: torch.Tensor, n_items: int, max_rows: int,
+                           block_tables: torch.Tensor, out: torch.Tensor, nh: int, scale: float,
+                           dc: DiffCombine, err: torch.Tensor, max_ctx: int = 0,
+                           variant: str = "auto", splits: int = 0) -> None:
+    """Differential attention of prompt portions on the tensor cores (bfloat16; sizes:
+    ``diff_attention_takes``); ``items`` as in ``prefill_attention``.  ``variant``: ``umma``
+    (tcgen05, d 64 and dv 128, page sizes 8..64 that divide 64), ``mma_sync``, or ``auto``:
+    the first where it applies.  ``max_ctx``: the longest context among the portions; few rows
+    after many cached keys then have their keys shared out over several CTAs of the umma
+    kernel (``splits`` forces a number)."""
+    global _launches
+    nkv, d, dv = _diff_check(q, k_cache, v_cache, out, nh, dc)
+    _want(items, torch.int32, "items")
+    if not diff_attention_takes(q.dtype, d, dv, scale, dc.temp_coef):
+        raise KernelError("differential attention: bfloat16, sizes multiples of 16 up to 128, a "
+                          "positive scale")
+    ps = k_cache.shape[2]
+    g = dc.gate
+    umma_ok = (d == 64 and dv == 128 and 8 <= ps <= 64 and 64 % ps == 0 and q.stride(0) % 8 == 0
+               and q.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+               and (g is None or (g.stride(0) % 8 == 0 and g.data_ptr() % 16 == 0)))
+    if variant not in ("auto", "umma", "mma_sync") or (variant == "umma" and not umma_ok):
+        raise KernelError(f"differential attention: variant {variant!r} does not apply")
+    if umma_ok and variant != "mma_sync":
+        blocks = -(-max_rows // 128) * nh * n_items
+        if splits <= 0:
+            splits = 1
+            if blocks * 2 <= num_sms(q.device):
+                splits = max(1, min(8, num_sms(q.device) // blocks, max_ctx // 1024))
+        part_o = part_ml = None
+        T = q.shape[0]
+        if splits > 1:
+            part_o = torch.empty((T, nh, 2, splits, dv), dtype=torch.float32, device=q.device)
+            part_ml = torch.empty((T, nh, 2, splits, 2), dtype=torch.float32, device=q.device)
+            _launches += 1          # two kernels: the shares and their merge
+        _run("diff_attention_prefill_umma", lib().bf_diff_attention_prefill_umma, _ptr(q),
+             _c_ll(q.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(items), _c_int(n_items),
+             _c_int(max_rows), _c_int(T), _ptr(block_tables), _c_int(block_tables.stride(0)),
+             _ptr(out), _c_int(nh), _c_int(nkv), _c_int(ps), _c_int(k_cache.shape[0]),
+             _c_float(scale), _c_int(splits), _ptr(part_o), _ptr(part_ml), _ptr(err),
+             *dc.args(q, out), _stream())
+        return
+    _run("diff_attention_prefill_mma", lib().bf_diff_attention_prefill_mma, _ptr(q),
+         _c_ll(q.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(items), _c_int(n_items),
+         _c_int(max_rows), _ptr(block_tables), _c_int(block_tables.stride(0)), _ptr(out),
+         _c_int(nh), _c_int(nkv), _c_int(d), _c_int(dv), _c_int(ps), _c_int(k_cache.shape[0]),
+         _c_float(scale), _ptr(err), *dc.args(q, out), _stream())
+
+
+def diff_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                          rows: Optional[torch.Tensor], n_rows: int, seq_of_token: torch.Tensor,
+                          positions: torch.Tensor, block_tables: torch.Tensor, out: torch.Tensor,
+                          nh: int, scale: float, dc: DiffCombine, max_ctx_len: int,
+                          err: torch.Tensor, variant: str = "auto") -> None:
+    """Differential attention of rows that bring one token each on the tensor cores (bfloat16;
+    sizes: ``diff_attention_takes``), ``rows`` and ``max_ctx_len`` as in ``decode_attention``.
+    ``variant``: ``persistent`` (resident CTAs and a ring of TMA-fed tiles; 2 d = dv = 64 or 128,
+    page sizes 8..128 that divide 128, at most 8 heads per kv head and 512 rows), ``mma_sync``,
+    or ``auto``: the first where it applies.  Shares of 128 keys leave partial results that a
+    merge kernel makes one, the two maps included."""
+    global _launches
+    nkv, d, dv = _diff_check(q, k_cache, v_cache, out, nh, dc)
+    if not diff_attention_takes(q.dtype, d, dv, scale, dc.temp_coef):
+        raise KernelError("differential attention: bfloat16, sizes multiples of 16 up to 128, a "
+                          "positive scale")
+    ps = k_cache.shape[2]
+    persistent_ok = (2 * d == dv and dv in (64, 128) and 8 <= ps <= 128 and 128 % ps == 0
+                     and nh // nkv <= 8 and n_rows <= 512 and q.stride(0) % 8 == 0
+                     and q.data_ptr() % 16 == 0)
+    if variant not in ("auto", "persistent", "mma_sync") or (variant == "persistent"
+                                                             and not persistent_ok):
+        raise KernelError(f"differential attention: variant {variant!r} does not apply")
+    splits = max(1, -(-int(max_ctx_len) // DECODE_SPLIT_KEYS))
+    part_o = torch.empty((n_rows, nh, 2, splits, dv), dtype=torch.float32, device=q.device)
+    part_ml = torch.empty((n_rows, nh, 2, splits, 2), dtype=torch.float32, device=q.device)
+    common = (_ptr(rows), _ptr(seq_of_token), _ptr(positions), _ptr(block_tables),
+              _c_int(block_tables.stride(0)), _ptr(out), _ptr(part_o), _ptr(part_ml),
+              _c_int(n_rows), _c_int(nh), _c_int(nkv))
+    tail = (_c_int(ps), _c_int(k_cache.shape[0]), _c_int(splits), _c_float(scale), _ptr(err),
+            *dc.args(q, out), _stream())
+    if persistent_ok and variant != "mma_sync":
+        _run("diff_attention_decode_persistent", lib().bf_diff_attention_decode_persistent,
+             _ptr(q), _c_ll(q.stride(0)), _ptr(k_cache), _ptr(v_cache), *common, _c_int(dv), *tail)
+    else:
+        _run("diff_attention_decode_mma", lib().bf_diff_attention_decode_mma, _ptr(q),
+             _c_ll(q.stride(0)), _ptr(k_cache), _ptr(v_cache), *common, _c_int(d), _c_int(dv),
+             *tail)
+    _launches += 1          # two kernels: the shares and their merge
+
+
 def sgemm_nt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     """out[M, N] = a[M, K] @ w[N, K]^T in true 32-bit arithmetic."""
     for t, n in ((a, "a"), (w, "w"), (out, "out")):

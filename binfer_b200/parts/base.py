@@ -141,9 +141,11 @@ class Norm(Part):
                 n_rows: int = 0) -> torch.Tensor:
         raise NotImplementedError
 
-    def add_normed(self, stream: "ResidualStream", y: torch.Tensor) -> None:
+    def add_normed(self, stream: "ResidualStream", y: torch.Tensor,
+                   next_norm: Optional["Norm"] = None) -> None:
         """``stream += norm(y)``: the norm on a sublayer's output (arrangements whose
-        sublayers read the stream itself).  Leaves ``stream.reading`` current."""
+        sublayers read the stream itself).  Leaves ``stream.reading`` current, or the output
+        of ``next_norm`` over the new stream in ``stream.ready``."""
         raise NotImplementedError
 
 
@@ -203,14 +205,15 @@ class ResidualStream:
     the stream while it normalises (one pass over memory instead of two).  Where a
     sublayer ends in a product and the kernels can do it, :meth:`add_linear` goes further:
     the product's epilogue adds into the stream and prepares the next norm's output, which
-    then waits in ``ready`` for that norm (``ready_for``).
+    then waits in ``ready`` for that norm (``ready_for``).  A norm on a sublayer's output can
+    leave the next norm's output there as well (``Norm.add_normed``).
     """
 
     def __init__(self, x: torch.Tensor):
         self.x = x
         self.pending: Optional[torch.Tensor] = None
         self.pending2: Optional[torch.Tensor] = None     # see add_pair
-        self.ready: Optional[ScaledRows] = None
+        self.ready = None                # a tensor, or ScaledRows
         self.ready_for = None
         # the stream itself in the activation type, for sublayers that read it without a
         # norm in front; kept by the kernel that last changed the stream, dropped by any other

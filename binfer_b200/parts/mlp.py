@@ -1,5 +1,6 @@
 """Dense gated feed-forward: ``down( act(gate(x)) * up(x) )``, ``act`` silu (SwiGLU) or the
-tanh form of gelu (``GatedMLPSpec.activation``; the products with the activation in their
+tanh form of gelu, or the clamped form ``min(g, c) sigmoid(a min(g, c)) (clamp(u, -c, c) + b)``
+with three constants (``GatedMLPSpec.activation``; the products with the activation in their
 epilogue are silu's, another activation runs the product and the activation kernel).
 
 ``silu(g) = g / (1 + exp(-g))`` (cuda/kernels/bf16_kernels.cu:461-477).  The
@@ -33,6 +34,8 @@ class GatedMLP(FeedForward):
             raise ValueError(f"activation {spec.activation!r} is not supported (supported: "
                              f"{sorted(ops.GATE_ACTIVATIONS)})")
         self.silu = spec.activation == "silu"
+        if spec.activation == "clamped" and not spec.limit > 0:
+            raise ValueError("a clamped activation needs a positive limit")
         if spec.bias:
             raise ValueError("feed-forward biases are not supported")
         self.spec, self.hidden, self.prefix, self.env = spec, hidden_size, prefix, env
@@ -68,7 +71,8 @@ class GatedMLP(FeedForward):
             if self.silu:
                 ops.silu_mul(gu, h, row_scale=row_scale)
             else:
-                ops.gated_act_mul(gu, h, self.spec.activation)
+                ops.gated_act_mul(gu, h, self.spec.activation, self.spec.limit,
+                                  self.spec.slope, self.spec.up_offset)
         return DeferredLinear(h, self.w_down)
 
     def _project_fused(self, x, h, row_scale) -> bool:

@@ -25,12 +25,14 @@ from .linear import linear
 
 # importing the modules registers the built-in parts
 from . import attention as _attention  # noqa: F401
+from . import attention_diff as _attention_diff  # noqa: F401
 from . import attention_latent as _attention_latent  # noqa: F401
 from . import attention_pooled as _attention_pooled  # noqa: F401
 from . import delta_rule as _delta_rule  # noqa: F401
 from . import mamba2 as _mamba2  # noqa: F401
 from . import block as _block          # noqa: F401
 from . import block_sublayer_norm as _block_sublayer_norm  # noqa: F401
+from . import block_sandwich as _block_sandwich  # noqa: F401
 from . import block_parallel as _block_parallel  # noqa: F401
 from . import attention_conv_window as _attention_conv_window  # noqa: F401
 from . import retention as _retention  # noqa: F401
@@ -54,6 +56,14 @@ class DecoderModel:
                           else ParamSpec(names.lm_head, (spec.vocab_size, spec.hidden_size)))
         self.embed: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
+        # frequencies of the vectors that positions add to the embedding output, one per pair
+        # of columns; double, so that the angle at a far position keeps its precision
+        self.position_freqs: Optional[torch.Tensor] = None
+        if spec.position_vectors is not None:
+            i = torch.arange((spec.hidden_size + 1) // 2, dtype=torch.float64)
+            self.position_freqs = torch.pow(
+                torch.tensor(spec.position_vectors.base, dtype=torch.float64),
+                -2.0 * i / spec.hidden_size).to(env.device)
         self.pass_spec = (None if spec.pass_table is None else
                           ParamSpec(spec.pass_table[0], (int(spec.pass_table[1]), spec.hidden_size),
                                     init="around_zero", role="vector"))
@@ -64,6 +74,10 @@ class DecoderModel:
                     and 0 <= entry.before.row < self.pass_spec.shape[0]):
                 raise ValueError(f"schedule entry {e} adds row {entry.before.row} of a table "
                                  f"of pass vectors that the model lacks or that is shorter")
+            if (entry.before is not None and entry.before.embedding
+                    and spec.position_vectors is not None):
+                raise ValueError("the embedding output cannot be added again where positions "
+                                 "add vectors to it")
             if not 0 <= entry.layer < len(self.blocks):
                 raise ValueError(f"schedule entry {e} names layer {entry.layer}, "
                                  f"but there are {len(self.blocks)} layers")
@@ -150,7 +164,9 @@ class DecoderModel:
         """Logits ``[R, vocab]`` (float32) at ``ctx.logit_rows``."""
         spec = self.spec
         resid = torch.empty((ctx.T, spec.hidden_size), dtype=torch.float32, device=self.env.device)
-        ops.embed_gather(self.embed, ctx.token_ids, resid, spec.embedding_scale, ctx.err)
+        ops.embed_gather(self.embed, ctx.token_ids, resid, spec.embedding_scale, ctx.err,
+                         ctx.positions if self.position_freqs is not None else None,
+                         self.position_freqs)
         stream = ResidualStream(resid)
         last = len(spec.schedule) - 1
         for e, entry in enumerate(spec.schedule):

@@ -19,7 +19,8 @@ choice only; the outputs may form groups of which only the best can be chosen fr
 chosen scores are divided by their sum and multiplied by a factor.  The router's last
 ``identity`` outputs stand for experts that return their input: they have no tensors, the
 router adds their weights up in one column, and a small kernel adds input times that column
-to the result.
+to the result.  A third way ("sigmoid") takes the sigmoids of the outputs as scores; a group may
+count by the sum of its few largest scores, and the chosen scores may stay as they are.
 
 A step of very few tokens in bfloat16 (a request that decodes alone) would read every expert
 for nothing; there the chosen experts' rows alone are read, a warp per output row
@@ -50,12 +51,12 @@ class MoEFeedForward(FeedForward):
         self.identity = int(getattr(spec, "identity", 0) or 0)
         if not 1 <= spec.top <= spec.num_experts + self.identity:
             raise ValueError("moe: top must be between 1 and the number of router outputs")
-        if spec.scoring not in ("softmax_top", "softmax_all"):
+        if spec.scoring not in ops.MOE_SCORINGS:
             raise ValueError(f"moe: unknown scoring {spec.scoring!r}")
         if spec.scoring == "softmax_top" and (self.identity or spec.groups > 1
-                                              or spec.correction):
-            raise ValueError("moe: corrections, groups and identity outputs go with the "
-                             "softmax over all outputs")
+                                              or spec.correction or not spec.normalize):
+            raise ValueError("moe: corrections, groups, identity outputs and scores that are "
+                             "not normalized go with scores over all outputs")
         n = spec.num_experts + self.identity
         if (spec.groups < 1 or n % spec.groups or not 1 <= spec.groups_keep <= spec.groups
                 or spec.top > spec.groups_keep * (n // spec.groups)):
@@ -120,7 +121,8 @@ class MoEFeedForward(FeedForward):
         ops.moe_route(x, self.w_router, self.E, self.top, self.gated_shared, route_w, top_ids,
                       top_w, scoring=s.scoring, correction=self.correction, groups=s.groups,
                       groups_keep=s.groups_keep, identity=self.identity,
-                      route_scale=s.route_scale, weight_eps=s.weight_eps)
+                      route_scale=s.route_scale, weight_eps=s.weight_eps,
+                      group_top=s.group_top, normalize=s.normalize)
         if (SPARSE and x.dtype == torch.bfloat16 and 2 * T * self.top <= self.E
                 and ops.moe_sparse_takes(self.hidden, self.ff, self.ff_sh, self.top)):
             # so few tokens that most experts are chosen by none: read the chosen ones alone

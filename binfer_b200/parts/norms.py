@@ -49,7 +49,7 @@ class RMSNorm(Norm):
         stream holds this norm's output already (``ResidualStream.add_linear``)."""
         if rows is None and stream.ready_for is self:
             out, stream.ready, stream.ready_for = stream.ready, None, None
-            return out           # ScaledRows: the product before already prepared this norm
+            return out           # the kernel before already prepared this norm
         if stream.pending2 is not None:
             stream.flush()       # a pair of adds: this norm's kernel folds one only
         stream.ready = stream.ready_for = None
@@ -62,15 +62,26 @@ class RMSNorm(Norm):
         return out
 
 
-    def add_normed(self, stream: ResidualStream, y: torch.Tensor) -> None:
+    def add_normed(self, stream: ResidualStream, y: torch.Tensor,
+                   next_norm: Optional[Norm] = None) -> None:
         """``stream.x += y * rsqrt(mean(y^2) + eps) * w`` in one kernel, which also leaves the
-        new stream in the activation type for the next sublayer's products."""
+        new stream in the activation type for the next sublayer's products, or, with
+        ``next_norm`` (the RMS norm that reads the stream next), that norm's output, which then
+        waits in ``stream.ready``."""
         stream.flush()
         stream.ready = stream.ready_for = None
         if y.dtype != self.env.dtype or y.shape != stream.x.shape:
             raise ValueError("add_normed: the sublayer's output must have the stream's shape "
                              "and the engine's activation type")
         reading = None
+        fs = getattr(next_norm, "fused_scale", None)
+        if fs is not None:
+            weight, eps = fs()
+            ready = torch.empty(stream.x.shape, dtype=self.env.dtype, device=self.env.device)
+            ops.rmsnorm_add(stream.x, y, self.weight, ready, self.eps, next_weight=weight,
+                            next_eps=eps)
+            stream.ready, stream.ready_for, stream.reading = ready, next_norm, None
+            return
         if self.env.dtype != torch.float32:
             reading = torch.empty(stream.x.shape, dtype=self.env.dtype, device=self.env.device)
         ops.rmsnorm_add(stream.x, y, self.weight, reading, self.eps)
