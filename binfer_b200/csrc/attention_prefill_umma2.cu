@@ -440,8 +440,9 @@ prefill_attention_umma2_kernel(const __grid_constant__ CUtensorMap map_q,
           if (__all_sync(0xffffffffu, mbar_wait(my_o_done + ((n - 1) & 1),
                                                 (uint32_t)((n - 1) >> 1) & 1u, abort))) {
             tc_fence_after();
-            const float f0 = factor[0] == 0.f ? 1.f : factor[0];   // 0: the row had nothing yet
-            const float f1 = factor[1] == 0.f ? 1.f : factor[1];
+            // (a factor of zero is right for a row that had nothing yet, whose O is zero, and
+            // for one whose maximum rose so far that what it had no longer counts)
+            const float f0 = factor[0], f1 = factor[1];
 #pragma unroll 1
             for (int c0 = 0; c0 < D; c0 += 64) {
               uint32_t w[32];

@@ -975,6 +975,32 @@ def test_prefill_attention_long_portions(cuda_device, ps, window, neighbours, va
     _close(out, ref, BF16)
 
 
+@pytest.mark.parametrize("far", [40, 70, 130, 200, 390])
+@pytest.mark.parametrize("variant", ["mma_sync", "umma", "umma2"])
+def test_prefill_attention_when_one_key_dwarfs_the_tiles_before_it(cuda_device, variant, far):
+    """A score hundreds above everything in earlier key tiles: what those tiles have left in the
+    output counts nothing any more (the factor on it underflows to zero)."""
+    from binfer_b200.csrc import ops
+    nh, nkv, d, ps, n = 4, 2, 128, 16, 400
+    g = torch.Generator().manual_seed(far)
+    q, k, v = (torch.randn(n, h, d, generator=g).to(BF16).double() for h in (nh, nkv, nkv))
+    k[far] = 0
+    k[far, :, 0] = 128.0
+    q[-1, :, 0] = 64.0                      # a score of 724
+    kc, vc, ids = _paged(k, v, ps, "cpu", BF16, 3)
+    ref = P.causal_attention(q, k, v, d ** -0.5, None).reshape(n, nh * d)
+    qd = q.to(BF16).reshape(n, nh * d).to(cuda_device)
+    bt = torch.tensor([ids], dtype=torch.int32, device=cuda_device)
+    items = torch.tensor([[0, 0, n, 0]], dtype=torch.int32, device=cuda_device)
+    out = torch.zeros_like(qd)
+    err = _err(cuda_device)
+    ops.prefill_attention(qd, kc.to(cuda_device), vc.to(cuda_device), items, 1, n, bt, out, nh,
+                          nkv, d, None, d ** -0.5, err, variant=variant)
+    assert int(err.item()) == 0
+    _close(out[-1:], ref[-1:], BF16)
+    _close(out, ref, BF16)
+
+
 @pytest.mark.parametrize("M,N,K,bn,c", [(1, 300, 520, 64, 4), (8, 4096, 4096, 128, 4),
                                         (16, 1000, 4104, 128, 8), (7, 6144, 4096, 192, 4),
                                         (3, 256, 256, 256, 2), (16, 4096, 12288, 128, 4),
