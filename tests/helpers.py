@@ -682,3 +682,95 @@ def make_folivik_dir(tmp_path, which, dtype=torch.float32, raw=None, tweak=None,
         tweak(w)
     save_file(w, os.path.join(d, "model.safetensors"))
     return d
+
+
+# ---------------------------------------------------- the design with differential attention
+def _pab_attn(heads, kv_heads, dim, vdim, diff=0.4, scale=None, temp=(0.25, 8), kv_from=None):
+    mx = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "diff": diff,
+          "scale": dim ** -0.5 if scale is None else scale}
+    if temp is not None:
+        mx["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    if kv_from is not None:
+        mx["kv_from"] = kv_from
+    return mx
+
+
+def _pab_dense(ff, limit):
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def _pab_moe(experts, top, ff, groups=None):
+    router = {"experts": experts, "top": top}
+    if groups is not None:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff}, "router": router}
+
+
+def _pab_layer(mixer, mlp=None):
+    return {"type": "attention", "mixer": mixer, "mlp": mlp}
+
+
+# two caches, the first read by two later layers around the second; a layer without a
+# feed-forward that reads another's cache; dense layers with two limits, mixtures with and
+# without groups; values larger and smaller than keys; two and one heads a key head
+PAB_A = {"architecture": "Pabelix", "vocab": 300, "width": 64, "norm": {"eps": 1e-5},
+         "layers": [_pab_layer(_pab_attn(4, 2, 16, 24, 0.3, 0.35), _pab_dense(96, 1.5)),
+                    _pab_layer(_pab_attn(4, 2, 16, 24, 0.6, 0.2, (0.5, 3), kv_from=0),
+                               _pab_moe(8, 3, 32, (4, 2))),
+                    _pab_layer(_pab_attn(2, 1, 24, 16, 0.8, 0.25, (0.4, 5)), _pab_moe(6, 2, 24)),
+                    _pab_layer(_pab_attn(2, 1, 24, 16, 0.5, kv_from=2)),
+                    _pab_layer(_pab_attn(4, 2, 16, 24, 0.1, kv_from=0), _pab_dense(40, 0.4))]}
+# a mixture first, whose groups are single experts; a key head for every query head; no query
+# temperature, and one that grows with every position; six heads on one key head; the last
+# layer reads the middle one
+PAB_B = {"architecture": "Pabelix", "vocab": 211, "width": 48, "norm": {"eps": 1e-6},
+         "layers": [_pab_layer(_pab_attn(3, 3, 8, 40, 0.2, temp=None), _pab_moe(5, 2, 40, (5, 3))),
+                    _pab_layer(_pab_attn(6, 1, 12, 8, 0.7, temp=(0.1, 1)), _pab_moe(9, 4, 16, (3, 2))),
+                    _pab_layer(_pab_attn(2, 2, 20, 20, 0.0, temp=(0.6, 64))),
+                    _pab_layer(_pab_attn(6, 1, 12, 8, 0.45, kv_from=1), _pab_dense(72, 3.0))]}
+# odd sizes everywhere: width, vocabulary, heads' sizes, inner features; one head; one expert
+PAB_C = {"architecture": "Pabelix", "vocab": 131, "width": 51, "norm": {"eps": 1e-5},
+         "layers": [_pab_layer(_pab_attn(1, 1, 7, 5, 0.5, 0.4), _pab_dense(13, 1.0)),
+                    _pab_layer(_pab_attn(3, 3, 10, 6, 0.3), _pab_moe(1, 1, 11)),
+                    _pab_layer(_pab_attn(1, 1, 7, 5, 0.9, kv_from=0), _pab_moe(4, 4, 9, (2, 2)))]}
+# wider, for bfloat16: sizes of the tcgen05 kernel (64 and 128), of the persistent decode
+# kernel alone (32 and 64) and of the mma.sync kernels alone
+PAB_D = {"architecture": "Pabelix", "vocab": 500, "width": 192, "norm": {"eps": 1e-5},
+         "layers": [_pab_layer(_pab_attn(4, 2, 64, 128, 0.4), _pab_dense(256, 2.5)),
+                    _pab_layer(_pab_attn(6, 3, 32, 64, 0.2, temp=(0.3, 20)), _pab_moe(8, 2, 64, (4, 2))),
+                    _pab_layer(_pab_attn(4, 2, 64, 128, 0.6, kv_from=0), _pab_moe(6, 3, 48)),
+                    _pab_layer(_pab_attn(5, 1, 80, 112, 0.5), _pab_dense(128, 1.0))]}
+
+PAB = {
+    "A": dict(raw=PAB_A, std=0.08, norm_std=0.15, page_size=16, seed=45),
+    "B": dict(raw=PAB_B, std=0.1, norm_std=0.15, page_size=4, seed=46),
+    "C": dict(raw=PAB_C, std=0.12, norm_std=0.15, page_size=8, seed=47),
+    "D": dict(raw=PAB_D, std=0.05, norm_std=0.1, page_size=16, seed=48),
+}
+
+
+def make_pabelix_dir(tmp_path, which, dtype=torch.float32, raw=None, tweak=None, tag="") -> str:
+    """A folder with config.json and random weights of a configuration of this design;
+    ``tweak(w)`` may change the tensors (a name -> tensor dictionary) before they are written."""
+    from binfer_b200.config import PabelixConfig
+    from binfer_b200.parts.model import param_specs_for
+    from binfer_b200.weights import random_tensors, save_file
+    t = PAB[which]
+    raw = raw or t["raw"]
+    cfg = PabelixConfig.from_dict(raw)
+    d = os.path.join(str(tmp_path), f"pab_{which}{tag}_{str(dtype).split('.')[-1]}")
+    os.makedirs(d, exist_ok=True)
+    with open(os.path.join(d, "config.json"), "w") as f:
+        json.dump(cfg.to_dict(), f)
+    w = random_tensors(param_specs_for(cfg.to_spec()), t["seed"], t["std"], t["norm_std"], dtype)
+    for n, x in w.items():
+        if n == "embed":                 # of the position vectors' order, so that both count
+            x *= 0.8 / t["std"]
+        elif n[-4:-1] in (".lq", ".lk"):  # lambda differs from layer to layer
+            x *= 3.0
+        elif n.endswith(("mlp.gate", "mlp.up")):   # the clamps are reached now and then
+            x *= 3.0
+    if tweak is not None:
+        tweak(w)
+    save_file(w, os.path.join(d, "model.safetensors"))
+    return d
