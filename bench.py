@@ -353,6 +353,25 @@ def state_space_config(size, layers=8):
             "layers": [pattern[i % 4] for i in range(layers)]}
 
 
+def differential_config(size, layers=8):
+    """The differential attention design at the Qwen3 shape of that name: the shape's query and
+    key heads, each of two maps of half the shape's head size (so that a token's keys and
+    values take as many bytes as the shape's) over values of its head size; every fourth layer
+    reads the keys and values of the layer two before it; the feed-forward is dense with the
+    shape's inner features in every other layer, else eight experts of a quarter of them in
+    four groups of which two are kept, two chosen."""
+    width, heads, kv, d, ff = HYBRID_SIZES[size][:5]
+    mixer = {"heads": heads, "kv_heads": kv, "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5,
+             "diff": 0.5, "q_temp": {"coef": 0.1, "every": 1024}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4},
+           "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Pabelix", "vocab": 32000, "width": width, "norm": {"eps": 1e-5},
+            "layers": [{"type": "attention", "mlp": moe if i % 2 else dense,
+                        "mixer": dict(mixer, kv_from=i - 2) if i % 4 == 3 else mixer}
+                       for i in range(layers)]}
+
+
 def hybrid_compare(args, design="hybrid"):
     """Prefill and decode throughput of the hybrid design (matrix-memory layers alternating
     with pooled-window attention layers), or with ``design`` "side_by_side" of the design
@@ -364,14 +383,16 @@ def hybrid_compare(args, design="hybrid"):
     (event pairs around every launch, eager).  Random weights, bfloat16."""
     import torch
     from binfer_b200 import Engine, Qwen3Config
-    from binfer_b200.config import FikotarConfig, FolivikConfig, GukidraConfig, KetopelConfig
+    from binfer_b200.config import (FikotarConfig, FolivikConfig, GukidraConfig, KetopelConfig,
+                                    PabelixConfig)
     from binfer_b200.engine.runner import StepItem
     from binfer_b200.profiling import Profiler
     layers = args.layers or 8
     B, context, ps = args.batch or 8, 4096, args.page_size
     steps, warmup = min(args.steps, 64), max(args.warmup, 3)
     what = {"hybrid": "hybrid design", "side_by_side": "side-by-side design",
-            "looped": "looped design", "state_space": "state space design"}[design]
+            "looped": "looped design", "state_space": "state space design",
+            "differential": "differential attention design"}[design]
     # the design with state space layers stands beside the looped design, the closest one
     # (latent attention, a recurrence per head, softmax attention), not beside Qwen3
     beside = "the looped design" if design == "state_space" else "the Qwen3 decoder"
@@ -387,6 +408,8 @@ def hybrid_compare(args, design="hybrid"):
                 else KetopelConfig.from_dict(looped_config(size, layers)) if design == "looped"
                 else FolivikConfig.from_dict(state_space_config(size, layers))
                 if design == "state_space"
+                else PabelixConfig.from_dict(differential_config(size, layers))
+                if design == "differential"
                 else FikotarConfig.from_dict(side_by_side_config(size, layers)))
         other = (("looped", KetopelConfig.from_dict(looped_config(size, layers)))
                  if design == "state_space" else ("qwen3", Qwen3Config.from_dict(qwen)))
@@ -540,8 +563,12 @@ def main():
                          "attention with a logarithmic distance bias and latent attention, with "
                          "a grouped router over experts and identity experts; it stands beside "
                          "the looped design instead of Qwen3")
-    ap.add_argument("--hybrid-sizes", default="", help="with --hybrid, --side-by-side, --looped or "
-                                                       "--state-space: 1.7b, 8b or both (default)")
+    ap.add_argument("--differential", action="store_true",
+                    help="the same for the design with differential attention, dense clamped "
+                         "feed-forwards and a mixture of experts with a sigmoid router")
+    ap.add_argument("--hybrid-sizes", default="",
+                    help="with --hybrid, --side-by-side, --looped, --state-space or "
+                         "--differential: 1.7b, 8b or both (default)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -558,6 +585,8 @@ def main():
         return hybrid_compare(args, "looped")
     if args.state_space:
         return hybrid_compare(args, "state_space")
+    if args.differential:
+        return hybrid_compare(args, "differential")
     if args.profile:
         return profile_steps(args)
     if args.workload == "serve":

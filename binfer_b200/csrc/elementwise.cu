@@ -8,6 +8,7 @@
 #include <stdlib.h>
 
 #include "common.cuh"
+#include "gate_act.cuh"
 
 static int g_pdl = -1;
 int bf_pdl_enabled() {
@@ -234,27 +235,7 @@ BF_EXPORT int bf_residual_add(float* resid, const void* delta, long long n, int 
 // out[t, c] = silu(gu[t, c]) * gu[t, I + c],  silu(g) = g / (1 + exp(-g))
 // (cuda/kernels/bf16_kernels.cu:461-477; there gate and up are separate buffers,
 // here they are the two halves of one fused projection's output row).
-// ACT 1: the tanh form of gelu in silu's place,
-//   gelu(g) = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
-// ACT 2: clamped, with three constants: g = min(gate, limit), u = clamp(up, -limit, limit),
-//   g sigmoid(slope g) (u + up_offset).
-#define BF_ACT_SILU 0
-#define BF_ACT_GELU_TANH 1
-#define BF_ACT_CLAMPED 2
-struct BfGateConst {
-  float limit, slope, up_offset;
-};
-template <int ACT>
-__device__ __forceinline__ float bf_gate_mul(float g, float u, const BfGateConst& k) {
-  if (ACT == BF_ACT_CLAMPED) {
-    g = fminf(g, k.limit);
-    u = fminf(fmaxf(u, -k.limit), k.limit) + k.up_offset;
-    return g / (1.f + expf(-k.slope * g)) * u;
-  }
-  if (ACT == BF_ACT_GELU_TANH)
-    return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-  return g / (1.f + expf(-g)) * u;
-}
+// ACT: the activations of gate_act.cuh.
 template <typename A, int ACT>
 __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, int T, int I,
                                 BfGateConst gk) {
@@ -267,25 +248,6 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, i
     const float u = bf_ld(gu + t * 2 * I + I + c);
     bf_st(out + i, bf_gate_mul<ACT>(g, u, gk));
   }
-}
-
-// silu for the bf16 kernels: float arithmetic with the hardware's exp2 and reciprocal
-// approximations (relative error about 2^-21, far inside the bf16 result's 2^-9).  With the
-// accurate expf and division the bf16 kernel was bound by arithmetic, not by memory.
-__device__ __forceinline__ float bf_silu_fast(float g) { return __fdividef(g, 1.f + __expf(-g)); }
-// ... and gelu's tanh form the same way: 0.5 g (1 + tanh(z)) = g / (1 + exp(-2 z))
-template <int ACT>
-__device__ __forceinline__ float bf_gate_mul_fast(float g, float u, const BfGateConst& k) {
-  if (ACT == BF_ACT_CLAMPED) {
-    g = fminf(g, k.limit);
-    u = fminf(fmaxf(u, -k.limit), k.limit) + k.up_offset;
-    return __fdividef(g, 1.f + __expf(-k.slope * g)) * u;
-  }
-  if (ACT == BF_ACT_GELU_TANH) {
-    const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-    return __fdividef(g, 1.f + __expf(-2.f * z)) * u;
-  }
-  return bf_silu_fast(g) * u;
 }
 
 // The same when the rows of gu still lack a factor (see BfRowScale).  I is at least 256, so

@@ -36,6 +36,7 @@
 #include <stdlib.h>
 
 #include "common.cuh"
+#include "gate_act.cuh"
 #include "tma_utils.cuh"
 #include "umma_utils.cuh"
 
@@ -87,10 +88,12 @@ struct ClusterGemmParams {
   // split of K): w is [2 inter, K], gate rows first; the tile's first bn/2 weight rows are
   // the gate rows of outputs tile * bn/2 .., the others the up rows of the same outputs, so
   // that one accumulator holds both; act_out[t, o] = silu(f g) * (f u), f the row's factor
-  // (rs), goes from tensor memory to global memory with no pass through shared memory.
+  // (rs), goes from tensor memory to global memory with no pass through shared memory.  The
+  // clamped activation (gate_act.cuh) with its constants `gk` is a form of its own.
   __nv_bfloat16* act_out;
   long long ldact;
   int inter;
+  BfGateConst gk;
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -177,11 +180,9 @@ __device__ __forceinline__ void load_weights(const ClusterGemmParams& p, const C
     tma_load_2d(dst + (size_t)h * BK * 2, map_w, bar, k, p.inter + tile * h);
   }
 }
-__device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.f + __expf(-g)); }
-
 // The epilogue's form is a template parameter, so that each instance carries only its own
-// code: with all four behind run-time tests the plain product was 3 % slower.
-enum { FORM_PLAIN = 0, FORM_ADD_NORM = 1, FORM_QKV = 2, FORM_SWIGLU = 3 };
+// code: with all of them behind run-time tests the plain product was 3 % slower.
+enum { FORM_PLAIN = 0, FORM_ADD_NORM = 1, FORM_QKV = 2, FORM_SWIGLU = 3, FORM_CLAMPED = 4 };
 
 constexpr int CL_THREADS = 256;       // eight warps: the roles of warps 1 to 3, then the epilogue
 
@@ -191,7 +192,8 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
                     const __grid_constant__ CUtensorMap map_w, OutT* __restrict__ out,
                     const ClusterGemmParams p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  constexpr bool kNorm = FORM == FORM_ADD_NORM, kQkv = FORM == FORM_QKV, kAct = FORM == FORM_SWIGLU;
+  constexpr bool kNorm = FORM == FORM_ADD_NORM, kQkv = FORM == FORM_QKV, kAct = FORM == FORM_SWIGLU || FORM == FORM_CLAMPED;
+  constexpr int kGate = FORM == FORM_CLAMPED ? BF_ACT_CLAMPED : BF_ACT_SILU;
   BF_TRACE_POINT(10 * BF_TR_GEMM);
   bf_pdl_trigger();
   uint8_t* base = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
@@ -384,10 +386,10 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
         uint32_t packed[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          const float a = silu_fast(__uint_as_float(g[2 * j]) * factor) *
-                          (__uint_as_float(u[2 * j]) * factor);
-          const float b = silu_fast(__uint_as_float(g[2 * j + 1]) * factor) *
-                          (__uint_as_float(u[2 * j + 1]) * factor);
+          const float a = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j]) * factor,
+                                                  __uint_as_float(u[2 * j]) * factor, p.gk);
+          const float b = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j + 1]) * factor,
+                                                  __uint_as_float(u[2 * j + 1]) * factor, p.gk);
           packed[j] = pack_bf16x2(__float_as_uint(a), __float_as_uint(b));
         }
         __nv_bfloat16* dst = p.act_out + (size_t)row * p.ldact + o0;
@@ -937,12 +939,16 @@ BF_EXPORT int bf_gemm_swiglu_plan(int inter, int K, int num_sms, int* bn_out) {
 // act[tokens, inter] = silu(f g) * (f u) with [g | u] = x[tokens, K] * w[2 inter, K]^T (gate
 // rows first) and f the factor of the norm before the projection (row_partials as in
 // bf_silu_mul_scaled; null: 1), as one kernel for at most 64 token rows.  bn from
-// bf_gemm_swiglu_plan.  Returns cudaErrorInvalidValue for what it does not take.
+// bf_gemm_swiglu_plan.  act_kind BF_ACT_CLAMPED: the clamped activation with its three constants
+// in silu's place.  Returns cudaErrorInvalidValue for what it does not take.
 BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int inter, int K,
                                   long long ldx, long long ldw, int bn, void* act,
                                   long long ldact, const float* row_partials, int row_count,
-                                  int row_width, float row_eps, int* err, cudaStream_t stream) {
+                                  int row_width, float row_eps, int* err, int act_kind,
+                                  float limit, float slope, float up_offset,
+                                  cudaStream_t stream) {
   if (tokens <= 0 || inter <= 0) return 0;
+  if (act_kind != BF_ACT_SILU && act_kind != BF_ACT_CLAMPED) return (int)cudaErrorInvalidValue;
   if (tokens > CL_MAX_TOKENS || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) ||
       ((uintptr_t)w & 15) || !act || ((uintptr_t)act & 15) || ldact % 8)
     return (int)cudaErrorInvalidValue;
@@ -961,6 +967,11 @@ BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int 
   p.rs.count = row_count;
   p.rs.inv_width = row_width > 0 ? 1.f / (float)row_width : 0.f;
   p.rs.eps = row_eps;
+  if (act_kind == BF_ACT_CLAMPED) {
+    p.gk = BfGateConst{limit, slope, up_offset};
+    return launch_cluster<__nv_bfloat16, FORM_CLAMPED>(x, w, (__nv_bfloat16*)nullptr, p, ldx, ldw,
+                                                        stream);
+  }
   return launch_cluster<__nv_bfloat16, FORM_SWIGLU>(x, w, (__nv_bfloat16*)nullptr, p, ldx, ldw,
                                                      stream);
 }

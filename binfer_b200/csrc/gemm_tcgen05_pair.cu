@@ -32,6 +32,7 @@
 #include <stdlib.h>
 
 #include "common.cuh"
+#include "gate_act.cuh"
 #include "tma_utils.cuh"
 #include "umma_utils.cuh"
 
@@ -47,6 +48,7 @@ struct PairParams {
   int accumulate;              // 1: out (float) += the product
   long long ldo;               // row stride of the output, in elements
   int* err;
+  BfGateConst gk;          // of the clamped activation (gated 2)
 };
 
 constexpr int PM = 256;                      // token rows per tile (128 per CTA)
@@ -107,7 +109,11 @@ __device__ __forceinline__ void pair_arrive_remote(uint32_t bar_cluster_addr) {
                    bar_cluster_addr)
                : "memory");
 }
-__device__ __forceinline__ float pair_silu(float g) { return __fdividef(g, 1.f + __expf(-g)); }
+// gated 1: silu(g) u; 2: the clamped activation
+__device__ __forceinline__ float pair_gate(float g, float u, int gated, const BfGateConst& gk) {
+  return gated == 2 ? bf_gate_mul_fast<BF_ACT_CLAMPED>(g, u, gk)
+                    : bf_gate_mul_fast<BF_ACT_SILU>(g, u, gk);
+}
 
 template <typename OutT>
 __device__ __forceinline__ void pair_store16(OutT* dst, const uint32_t (&r)[16], bool vec,
@@ -321,8 +327,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
                 tmem_ld32(taddr + col + 64, up);
 #pragma unroll
                 for (int j = 0; j < 32; ++j)
-                  r[j] = __float_as_uint(pair_silu(__uint_as_float(r[j])) *
-                                         __uint_as_float(up[j]));
+                  r[j] = __float_as_uint(pair_gate(__uint_as_float(r[j]), __uint_as_float(up[j]),
+                                                   p.gated, p.gk));
               }
 #pragma unroll
               for (int q = 0; q < 4; ++q) {
@@ -377,8 +383,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
               if (t < p.tokens && o0 < p.features) {
 #pragma unroll
                 for (int j = 0; j < 16; ++j)
-                  g[j] = __float_as_uint(pair_silu(__uint_as_float(g[j])) *
-                                         __uint_as_float(up[j]));
+                  g[j] = __float_as_uint(pair_gate(__uint_as_float(g[j]), __uint_as_float(up[j]),
+                                                   p.gated, p.gk));
                 pair_store16(out + (size_t)t * p.ldo + o0, g, vec_ok, p.features - o0, false);
               }
             }
@@ -517,14 +523,15 @@ BF_EXPORT int bf_gemm_pair_choose_bn(int tokens, int columns, int step, int num_
 
 // out[tokens, features] = x[tokens, K] * w[features, K]^T in bf16 with float accumulation, on
 // pairs of CTAs.  gated != 0: w is [2 features, K] (gate rows first) and out[t, o] =
-// silu(x . w[o]) * (x . w[features + o]), bf16 only.  out_dtype: BF_DTYPE_BF16 or
+// silu(x . w[o]) * (x . w[features + o]), bf16 only; gated == 2: the clamped activation of
+// gate_act.cuh with its three constants instead.  out_dtype: BF_DTYPE_BF16 or
 // BF_DTYPE_F32.  accumulate != 0 (float out only): out += the product.  bn: accumulator
 // columns per tile (0: chosen here).  Returns
 // cudaErrorInvalidValue for shapes it does not take.
 BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tokens, int features,
                                 int K, long long ldx, long long ldw, long long ldo, int out_dtype,
                                 int gated, int accumulate, int bn, int num_sms, int* err,
-                                cudaStream_t stream) {
+                                float limit, float slope, float up_offset, cudaStream_t stream) {
   if (tokens <= 0 || features <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || num_sms < 2)
     return (int)cudaErrorInvalidValue;
@@ -541,7 +548,8 @@ BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tok
   p.K = K;
   p.ldo = ldo;
   p.bn = bn;
-  p.gated = gated ? 1 : 0;
+  p.gated = gated == 2 ? 2 : (gated ? 1 : 0);
+  p.gk = BfGateConst{limit, slope, up_offset};
   p.accumulate = accumulate ? 1 : 0;
   p.tiles_t = (tokens + PM - 1) / PM;
   p.tiles_f = (columns + bn - 1) / bn;

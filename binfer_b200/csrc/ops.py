@@ -192,6 +192,7 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor,
 
 
 GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
+FUSED_ACTIVATIONS = ("silu", "clamped")     # those that a product applies in its epilogue
 
 
 def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str,
@@ -1608,15 +1609,20 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Te
 
 
 def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Tensor,
-                   bn: int = 0, gated: bool = False, accumulate: bool = False) -> bool:
+                   bn: int = 0, gated: bool = False, accumulate: bool = False,
+                   activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
+                   up_offset: float = 0.0) -> bool:
     """out[M, N] = x[M, K] @ w[N, K]^T on pairs of SMs (``tcgen05.mma.cta_group::2``, tiles of
     256 token rows): the product for many token rows.  ``gated``: ``w`` is the stacked
     ``[2 N, K]`` gate/up weight and ``out[M, N] = silu(x w_gate^T) * (x w_up^T)``, bfloat16
-    only.  ``accumulate``: ``out`` (float32) ``+=`` the product.  ``bn``: accumulator columns
+    only; ``activation`` "clamped" with its constants as in ``gated_act_mul`` in silu's place.
+    ``accumulate``: ``out`` (float32) ``+=`` the product.  ``bn``: accumulator columns
     per tile (0: chosen by the library).  Returns False, having done nothing, for shapes the
     kernel does not take."""
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_bf16_pair: operands must be bfloat16")
+    if activation not in FUSED_ACTIVATIONS:
+        raise KernelError(f"gemm_bf16_pair: activation {activation!r} is not supported")
     if accumulate and (gated or out.dtype != torch.float32):
         raise KernelError("gemm_bf16_pair: accumulate needs a float32 output and no gate")
     M, K = x.shape
@@ -1629,8 +1635,10 @@ def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: tor
         return False
     _run("gemm_bf16_pair", lib().bf_gemm_bf16_pair, _ptr(x), _ptr(w), _ptr(out), _c_int(M),
          _c_int(N), _c_int(K), _c_ll(x.stride(0)), _c_ll(w.stride(0)), _c_ll(out.stride(0)),
-         _c_int(_dtype_code(out)), _c_int(1 if gated else 0), _c_int(1 if accumulate else 0),
-         _c_int(bn), _c_int(num_sms(x.device)), _ptr(err), _stream())
+         _c_int(_dtype_code(out)),
+         _c_int((2 if activation == "clamped" else 1) if gated else 0),
+         _c_int(1 if accumulate else 0), _c_int(bn), _c_int(num_sms(x.device)), _ptr(err),
+         _c_float(limit), _c_float(slope), _c_float(up_offset), _stream())
     return True
 
 
@@ -1754,10 +1762,15 @@ def gemm_swiglu_plan(inter: int, K: int, device: torch.device):
 
 
 def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor,
-                     err: torch.Tensor, bn: int, row_scale: Optional[RowScale] = None) -> bool:
+                     err: torch.Tensor, bn: int, row_scale: Optional[RowScale] = None,
+                     activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
+                     up_offset: float = 0.0) -> bool:
     """``silu_mul(x @ w_gate_up^T)`` as one kernel for at most 64 token rows: ``w_gate_up`` is
-    ``[2 I, K]`` with the gate rows first, ``out`` is ``[M, I]``.  Returns False, having done
+    ``[2 I, K]`` with the gate rows first, ``out`` is ``[M, I]``.  ``activation`` "clamped" with its
+    constants as in ``gated_act_mul`` in silu's place.  Returns False, having done
     nothing, for what the kernel does not take."""
+    if activation not in FUSED_ACTIVATIONS:
+        raise KernelError(f"gemm_bf16_swiglu: activation {activation!r} is not supported")
     M, K = x.shape
     I = out.shape[1]
     if (M > CLUSTER_MAX_TOKENS or K % 8 or x.stride(1) != 1 or w_gate_up.stride(1) != 1
@@ -1768,7 +1781,9 @@ def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor
         return False
     _run("gemm_bf16_swiglu", lib().bf_gemm_bf16_swiglu, _ptr(x), _ptr(w_gate_up), _c_int(M),
          _c_int(I), _c_int(K), _c_ll(x.stride(0)), _c_ll(w_gate_up.stride(0)), _c_int(bn),
-         _ptr(out), _c_ll(out.stride(0)), *_row_scale_args(row_scale, M), _ptr(err), _stream())
+         _ptr(out), _c_ll(out.stride(0)), *_row_scale_args(row_scale, M), _ptr(err),
+         _c_int(GATE_ACTIVATIONS[activation]), _c_float(limit), _c_float(slope),
+         _c_float(up_offset), _stream())
     return True
 
 

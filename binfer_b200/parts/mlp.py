@@ -1,7 +1,7 @@
 """Dense gated feed-forward: ``down( act(gate(x)) * up(x) )``, ``act`` silu (SwiGLU) or the
 tanh form of gelu, or the clamped form ``min(g, c) sigmoid(a min(g, c)) (clamp(u, -c, c) + b)``
-with three constants (``GatedMLPSpec.activation``; the products with the activation in their
-epilogue are silu's, another activation runs the product and the activation kernel).
+with three constants (``GatedMLPSpec.activation``; silu and the clamped form run in the products'
+epilogues where those kernels apply, else the product and the activation kernel run).
 
 ``silu(g) = g / (1 + exp(-g))`` (cuda/kernels/bf16_kernels.cu:461-477).  The
 reference runs gate and up as two products (src/engine/batched_engine.ts:1243-1244);
@@ -34,6 +34,9 @@ class GatedMLP(FeedForward):
             raise ValueError(f"activation {spec.activation!r} is not supported (supported: "
                              f"{sorted(ops.GATE_ACTIVATIONS)})")
         self.silu = spec.activation == "silu"
+        self.fusable = spec.activation in ops.FUSED_ACTIVATIONS
+        self._act = dict(activation=spec.activation, limit=spec.limit, slope=spec.slope,
+                         up_offset=spec.up_offset)
         if spec.activation == "clamped" and not spec.limit > 0:
             raise ValueError("a clamped activation needs a positive limit")
         if spec.bias:
@@ -71,20 +74,20 @@ class GatedMLP(FeedForward):
             if self.silu:
                 ops.silu_mul(gu, h, row_scale=row_scale)
             else:
-                ops.gated_act_mul(gu, h, self.spec.activation, self.spec.limit,
-                                  self.spec.slope, self.spec.up_offset)
+                ops.gated_act_mul(gu, h, **self._act)
         return DeferredLinear(h, self.w_down)
 
     def _project_fused(self, x, h, row_scale) -> bool:
         """Few token rows in bfloat16: the stacked projection with the activation in its
         epilogue, one CTA a tile of gate rows and the up rows of the same outputs.  False,
         having done nothing, where that kernel does not run."""
-        if not FUSE_SWIGLU or not self.silu or x.dtype != torch.bfloat16 or self.inter % 8:
+        if not FUSE_SWIGLU or not self.fusable or x.dtype != torch.bfloat16 or self.inter % 8:
             return False
         pair_from = pair_token_limit()
         if pair_from and x.shape[0] >= pair_from and row_scale is None:
             # many token rows: the product on pairs of SMs, the activation in its epilogue
-            return ops.gemm_bf16_pair(x, self.w_gate_up, h, ops.error_word(x.device), gated=True)
+            return ops.gemm_bf16_pair(x, self.w_gate_up, h, ops.error_word(x.device), gated=True,
+                                      **self._act)
         if x.shape[0] > swiglu_token_limit():
             return False
         if self._swiglu_plan is None:
@@ -93,7 +96,7 @@ class GatedMLP(FeedForward):
         if not plan or plan[1] < FUSE_SWIGLU_FILL * ops.num_sms(x.device):
             return False
         return ops.gemm_bf16_swiglu(x, self.w_gate_up, h, ops.error_word(x.device), plan[0],
-                                    row_scale=row_scale)
+                                    row_scale=row_scale, **self._act)
 
 
 register_ffn("gated_mlp", GatedMLP)

@@ -112,6 +112,36 @@ def test_norm_of_an_output_with_the_next_norm(cuda_device, dtype, width):
         assert H.rel_err(out.float().cpu(), want) <= (2e-6 if dtype == torch.float32 else 6e-3)
 
 
+@pytest.mark.parametrize("tokens,inner,width", [(1, 2048, 256), (8, 3072, 512), (64, 2560, 264),
+                                                (300, 512, 256), (1100, 520, 256)])
+def test_products_with_the_clamped_activation(cuda_device, tokens, inner, width):
+    """The stacked product with the activation in its epilogue, for few tokens and for many: the
+    same as the product followed by the activation, within the rounding of what lies between."""
+    from binfer_b200.csrc import ops
+    g = torch.Generator().manual_seed(tokens)
+    x = torch.randn(tokens, width, generator=g).to(BF16)
+    w = (torch.randn(2 * inner, width, generator=g) * 2 / width ** 0.5).to(BF16)
+    limit = 1.25
+    eye = torch.eye(inner, dtype=F64)
+    want = P.clamped_mlp(x.double(), {"f.gate": w[:inner].double(), "f.up": w[inner:].double(),
+                                      "f.down": eye}, "f.", limit)
+    out = torch.empty(tokens, inner, dtype=BF16, device=cuda_device)
+    k = dict(activation="clamped", limit=limit, slope=1.702, up_offset=1.0)
+    xd, wd, err = x.to(cuda_device), w.to(cuda_device), ops.error_word(cuda_device)
+    ran = 0
+    if tokens <= 64:
+        plan = ops.gemm_swiglu_plan(inner, width, cuda_device)
+        assert plan and ops.gemm_bf16_swiglu(xd, wd, out, err, plan[0], **k)
+        assert H.rel_err(out.float().cpu(), want) <= 6e-3
+        ran += 1
+    if tokens >= 64:
+        out.zero_()
+        assert ops.gemm_bf16_pair(xd, wd, out, err, gated=True, **k)
+        assert H.rel_err(out.float().cpu(), want) <= 6e-3
+        ran += 1
+    assert ran and int(err.item()) == 0
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, BF16], ids=["f32", "bf16"])
 @pytest.mark.parametrize("inner,limit", [(64, 1.5), (13, 0.3), (256, 7.0)])
 def test_clamped_activation(cuda_device, dtype, inner, limit):
