@@ -74,16 +74,6 @@ __device__ __forceinline__ bool dp_group_all(int id, int threads, bool ok) {
       : "memory");
   return r != 0;
 }
-// Untiled bulk copy global -> shared; both addresses 16-byte aligned, bytes a multiple of 16.
-__device__ __forceinline__ void dp_bulk_load(void* smem_dst, const void* src, uint32_t bytes,
-                                             uint64_t* bar) {
-  asm volatile(
-      "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::
-          "r"(bf_smem_u32(smem_dst)),
-      "l"(src), "r"(bytes), "r"(bf_smem_u32(bar))
-      : "memory");
-}
-
 struct DpSmem {
   size_t bars, qbuf, pbuf, red, info, row_start, row_t, row_p, row_seq, total;
 };
@@ -271,7 +261,7 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
           int* inf = info + e * 8;
           if (inf[7]) {
             inf[7] = 0;
-            dp_bulk_load(qbuf + (size_t)e * GQ * D,
+            bf_bulk_load(qbuf + (size_t)e * GQ * D,
                          q + (size_t)inf[5] * q_stride + (size_t)inf[1] * GQ * D,
                          (uint32_t)(GQ * D * 2), full + inf[6]);
           }
@@ -328,7 +318,7 @@ decode_attention_persistent_kernel(const __grid_constant__ CUtensorMap map_k,
             inf[0] = r; inf[1] = g; inf[2] = split;
             bf_mbar_expect_tx(full + slot, TILE_BYTES + (uint32_t)(GQ * D * 2));
             if (waited) {
-              dp_bulk_load(qbuf + (size_t)qi * GQ * D,
+              bf_bulk_load(qbuf + (size_t)qi * GQ * D,
                            q + (size_t)t * q_stride + (size_t)g * GQ * D,
                            (uint32_t)(GQ * D * 2), full + slot);
             } else {

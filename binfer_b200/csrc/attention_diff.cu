@@ -216,20 +216,23 @@ BF_EXPORT int bf_diff_attention_generic(
 }
 
 // --------------------------------------------------------------- shares of the keys made one
-// A block of 256 threads per (row, head): half m sums map m's shares in ascending order, each
-// with its weight, a column a thread; then the two maps become the head's output.
-#define DM_HALF 128
+// A block of eight warps per (row, head), four per map: a warp sums every fourth share of its
+// map, a lane four neighbouring columns, eight shares' loads in flight before anything else is
+// known; the four sums are then added in order and the two maps become the head's output.
+#define DM_WARPS 4
+#define DM_AHEAD 8
 
-__global__ void __launch_bounds__(2 * DM_HALF) diff_merge_kernel(
+__global__ void __launch_bounds__(2 * DM_WARPS * 32) diff_merge_kernel(
     const float* __restrict__ part_o, const float* __restrict__ part_ml,
     const int* __restrict__ rows, const int* __restrict__ positions,
     const int* __restrict__ items, __nv_bfloat16* __restrict__ out, int nh, int dv,
     int max_splits, int fixed, long long out_stride, BfDiffArgs dd) {
-  extern __shared__ float sh[];            // [2][max_splits] weights, [2][dv] the maps' outputs
+  extern __shared__ __align__(16) float sh[];   // [2][4][dv] the warps' sums, [2][max_splits] weights
   __shared__ float scratch[33];
   bf_pdl_trigger();
   bf_pdl_wait();
-  const int h = blockIdx.y, mp = threadIdx.x / DM_HALF, tid = threadIdx.x % DM_HALF;
+  const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int mp = warp / DM_WARPS, wm = warp % DM_WARPS;
   int r, t, n;
   if (items) {                             // a portion's row; its partials lie by token row
     const int* it = items + 4 * blockIdx.z;
@@ -241,47 +244,72 @@ __global__ void __launch_bounds__(2 * DM_HALF) diff_merge_kernel(
     t = rows ? rows[r] : r;
     n = min(max_splits, positions[t] / 128 + 1);
   }
-  float* wgt = sh + (size_t)mp * max_splits;
-  float* a = sh + (size_t)2 * max_splits;
+  float* sums = sh + (size_t)mp * DM_WARPS * dv;
+  float* wgt = sh + (size_t)2 * DM_WARPS * dv + (size_t)mp * max_splits;
   const size_t at = (((size_t)r * nh + h) * 2 + mp) * max_splits;
-  // every warp works the weights of its map out for itself as far as the maximum and the sum
-  // go (one round of loads, shuffles instead of barriers); the half's threads share the weights
-  const int lane = threadIdx.x & 31;
-  float M = -INFINITY;
-  for (int s = lane; s < n; s += 32) M = fmaxf(M, part_ml[(at + s) * 2]);
+  const float4* po = reinterpret_cast<const float4*>(part_o + at * dv);
+  const int dv4 = dv >> 2;
+  float4 x[DM_AHEAD];                      // the first shares of the lane's first columns
+#pragma unroll
+  for (int u = 0; u < DM_AHEAD; ++u) {
+    const int s = wm + DM_WARPS * u;
+    x[u] = s < n && lane < dv4 ? po[(size_t)s * dv4 + lane] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // every warp works out the maximum and the sum of its map; the map's first writes the weights
+  const float2* ml = reinterpret_cast<const float2*>(part_ml) + at;
+  const float2 mine = lane < n ? ml[lane] : make_float2(-INFINITY, 0.f);
+  float M = mine.x;
+  for (int s = lane + 32; s < n; s += 32) M = fmaxf(M, ml[s].x);
   M = warp_max(M);
-  float L = 0.f;
-  for (int s = lane; s < n; s += 32) {
-    const float ms = part_ml[(at + s) * 2];
-    if (ms != -INFINITY) L += part_ml[(at + s) * 2 + 1] * exp2f(ms - M);
-  }
+  float L = mine.x == -INFINITY ? 0.f : mine.y * exp2f(mine.x - M);
+  for (int s = lane + 32; s < n; s += 32)
+    if (ml[s].x != -INFINITY) L += ml[s].y * exp2f(ml[s].x - M);
   L = warp_sum(L);
-  const float inv = L > 0.f ? 1.f / L : 0.f;
-  for (int s = tid; s < n; s += DM_HALF) {
-    const float ms = part_ml[(at + s) * 2];
-    wgt[s] = ms == -INFINITY ? 0.f : exp2f(ms - M) * inv;
-  }
-  __syncthreads();
-  for (int c = tid; c < dv; c += DM_HALF) {
-    float v = 0.f;
-    const float* po = part_o + at * dv + c;
-    int s = 0;
-    for (; s + 8 <= n; s += 8) {           // eight loads in flight, added in order
-      float x[8];
-#pragma unroll
-      for (int u = 0; u < 8; ++u) x[u] = wgt[s + u] != 0.f ? po[(size_t)(s + u) * dv] : 0.f;
-#pragma unroll
-      for (int u = 0; u < 8; ++u) v += x[u] * wgt[s + u];
+  if (wm == 0) {
+    const float inv = L > 0.f ? 1.f / L : 0.f;
+    for (int s = lane; s < n; s += 32) {
+      const float ms = s < 32 ? mine.x : ml[s].x;
+      wgt[s] = ms == -INFINITY ? 0.f : exp2f(ms - M) * inv;
     }
-    for (; s < n; ++s)
-      if (wgt[s] != 0.f) v += po[(size_t)s * dv] * wgt[s];
-    a[mp * dv + c] = v;
   }
   __syncthreads();
+  for (int c = lane; c < dv4; c += 32) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s0 = wm; s0 < n; s0 += DM_WARPS * DM_AHEAD) {
+      if (s0 != wm || c != lane) {
+#pragma unroll
+        for (int u = 0; u < DM_AHEAD; ++u) {
+          const int s = s0 + DM_WARPS * u;
+          if (s < n) x[u] = po[(size_t)s * dv4 + c];
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < DM_AHEAD; ++u) {
+        const int s = s0 + DM_WARPS * u;
+        const float w = s < n ? wgt[s] : 0.f;
+        if (w != 0.f) {                    // (a share without keys has left nothing)
+          v.x += x[u].x * w;
+          v.y += x[u].y * w;
+          v.z += x[u].z * w;
+          v.w += x[u].w * w;
+        }
+      }
+    }
+    reinterpret_cast<float4*>(sums + (size_t)wm * dv)[c] = v;
+  }
+  __syncthreads();
+  float* a1 = sh;
+  const float* a2 = sh + (size_t)DM_WARPS * dv;
   float ss = 0.f;
-  for (int c = threadIdx.x; c < dv; c += 2 * DM_HALF) {
-    const float o = a[c] - dd.lambda * a[dv + c];
-    a[c] = o;
+  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
+    float o1 = 0.f, o2 = 0.f;
+#pragma unroll
+    for (int w = 0; w < DM_WARPS; ++w) {
+      o1 += a1[w * dv + c];
+      o2 += a2[w * dv + c];
+    }
+    const float o = o1 - dd.lambda * o2;
+    a1[c] = o;                             // (this thread's own column)
     ss += o * o;
   }
   ss = block_sum(ss, scratch);
@@ -290,8 +318,8 @@ __global__ void __launch_bounds__(2 * DM_HALF) diff_merge_kernel(
   const __nv_bfloat16* gate =
       dd.gate ? (const __nv_bfloat16*)dd.gate + (size_t)t * dd.gate_stride + (size_t)h * dv
               : nullptr;
-  for (int c = threadIdx.x; c < dv; c += 2 * DM_HALF) {
-    float v = a[c] * f;
+  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
+    float v = a1[c] * f;
     if (gate) v *= bf_sigmoid_fast(__bfloat162float(gate[c]));
     o[c] = __float2bfloat16_rn(v);
   }
@@ -301,8 +329,9 @@ static int diff_merge(dim3 grid, const float* part_o, const float* part_ml, cons
                       const int* positions, const int* items, void* out, int nh, int dv,
                       int max_splits, int fixed, long long out_stride, const BfDiffArgs& dd,
                       cudaStream_t stream) {
-  const size_t smem = (size_t)2 * (max_splits + dv) * sizeof(float);
-  if (smem > 200 * 1024 || dv <= 0 || max_splits <= 0) return (int)cudaErrorInvalidValue;
+  const size_t smem = (size_t)2 * (max_splits + DM_WARPS * dv) * sizeof(float);
+  if (smem > 200 * 1024 || dv <= 0 || dv % 4 || max_splits <= 0 || ((uintptr_t)part_o & 15) ||
+      ((uintptr_t)part_ml & 7)) return (int)cudaErrorInvalidValue;
   if (smem > 48 * 1024) {
     static size_t configured[BF_MAX_DEVICES];
     size_t& c = configured[bf_current_device()];
@@ -313,7 +342,7 @@ static int diff_merge(dim3 grid, const float* part_o, const float* part_ml, cons
       c = 200 * 1024;
     }
   }
-  return bf_launch_pdl(diff_merge_kernel, grid, dim3(2 * DM_HALF), smem, stream, part_o, part_ml,
+  return bf_launch_pdl(diff_merge_kernel, grid, dim3(2 * DM_WARPS * 32), smem, stream, part_o, part_ml,
                        rows, positions, items, (__nv_bfloat16*)out, nh, dv, max_splits, fixed,
                        out_stride, dd);
 }

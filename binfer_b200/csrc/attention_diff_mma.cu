@@ -10,9 +10,10 @@
 // both maps' O += P V.  A row's values lie in the four lanes of a quad, so the epilogue
 // (difference, root mean square, gate) needs two shuffles.
 //
-// Single tokens: a warp takes one share of 128 keys (four tiles of 32) for up to 16 heads of a
-// group and leaves a partial result per map for the merge kernel; the four warps of a CTA take
-// neighbouring shares and never wait for each other.
+// Single tokens: a warp takes one share of 128 keys for up to 16 heads of a group and leaves a
+// partial result per map for the merge kernel; the four warps of a CTA take neighbouring shares
+// and never wait for each other.  A warp's tiles of 16 keys come by bulk copies, a row a lane (16
+// key rows, 16 value rows), three tiles under way; two CTAs fit an SM.
 //
 // q is read from the rows of the stacked projection; the query temperature rides on the scale.
 #include <float.h>
@@ -20,12 +21,14 @@
 #include "attention_diff.cuh"
 #include "common.cuh"
 #include "mma_utils.cuh"
+#include "tma_utils.cuh"
 
 #define DA_ROWS 64
 #define DA_KEYS 64
 #define DA_THREADS 128
 #define DA_SHARE 128        // keys a warp takes while decoding
-#define DA_DKEYS 32         // ... in tiles of this many
+#define DA_DKEYS 16         // ... in tiles of this many
+#define DA_DSTAGES 3        // ... of which this many are under way
 
 __device__ __forceinline__ float da_ex2(float x) {
   float y;
@@ -33,19 +36,39 @@ __device__ __forceinline__ float da_ex2(float x) {
   return y;
 }
 
-// `rows` cache rows of d elements on their way into a shared tile, by `nthreads` threads (thread
-// `id`): row r is the cache's row where[r] (-1: none, the tile's row is zeroed).
+// A walk over the 16-byte pieces of a tile's rows by `n` threads: the piece of this thread at
+// first and the step to its next one, so that the loop divides nothing.
+struct DaWalk {
+  int row, c, chunks, drow, dc;
+};
+__device__ __forceinline__ DaWalk da_walk(int d, int id, int n) {
+  DaWalk w;
+  w.chunks = d >> 3;
+  w.row = id / w.chunks;
+  w.c = id - w.row * w.chunks;
+  w.drow = n / w.chunks;
+  w.dc = n - w.drow * w.chunks;
+  return w;
+}
+// `rows` cache rows on their way into a shared tile: tile row r is the cache's row at(r) (-1:
+// none, the tile's row is zeroed: a copy of 0 bytes reads nothing).  Every thread of a warp
+// makes as many steps as any other (`at` may be a shuffle).
+template <typename AtFn>
 __device__ __forceinline__ void da_load_rows(__nv_bfloat16* tile, int pitch,
-                                             const __nv_bfloat16* __restrict__ cache,
-                                             const int* where, int rows, int d, int id,
-                                             int nthreads) {
-  const int chunks = d >> 3;
-  for (int i = id; i < rows * chunks; i += nthreads) {
-    const int r = i / chunks, c = (i - r * chunks) << 3;
-    const int at = where[r];
-    // (0 bytes: nothing is read, the 16 bytes are zeroed)
-    cp_async16(tile + (size_t)r * pitch + c, at >= 0 ? cache + (size_t)at * d + c : cache,
-               at >= 0 ? 16 : 0);
+                                             const __nv_bfloat16* __restrict__ cache, int rows,
+                                             DaWalk w, int steps, AtFn at) {
+#pragma unroll 4
+  for (int k = 0; k < steps; ++k) {
+    const int e = at(min(w.row, rows - 1));
+    if (w.row < rows)
+      cp_async16(tile + w.row * pitch + w.c * 8,
+                 cache + (e >= 0 ? ((size_t)e * w.chunks + w.c) * 8 : 0), e >= 0 ? 16 : 0);
+    w.row += w.drow;
+    w.c += w.dc;
+    if (w.c >= w.chunks) {
+      w.c -= w.chunks;
+      ++w.row;
+    }
   }
 }
 // The cache row of key e of a request for kv head g, or -1 beyond `limit` (or a bad page).
@@ -106,7 +129,10 @@ __device__ __forceinline__ void da_scores(const __nv_bfloat16* qt, int pitch_q,
   for (int i = 0; i < 2; ++i) {
     mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
     mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-    const float m_new = fmaxf(m[i], mx[i] * sc[i]);      // the factor is positive
+    // the reference follows the maximum only when that has grown by more than 8 (a factor of
+    // 256 in the probabilities, harmless in bfloat16 and float), so O is rarely rescaled
+    const float top = mx[i] * sc[i];                     // the factor is positive
+    const float m_new = top > m[i] + 8.f ? top : m[i];
     ref[i] = m_new == -INFINITY ? 0.f : m_new;           // a row that has seen nothing yet
     corr[i] = da_ex2(m[i] - ref[i]);
     m[i] = m_new;
@@ -133,13 +159,17 @@ template <int KT, int DVT>
 __device__ __forceinline__ void da_values(const __nv_bfloat16* vt, int pitch_v, int dv, int lane,
                                           const uint32_t (&pa)[2][KT / 16][4],
                                           const float (&corr)[2][2], float (&o)[2][DVT][4]) {
+  // (most tiles move no row's reference: the factors are one)
+  if (__any_sync(0xffffffffu, corr[0][0] != 1.f || corr[0][1] != 1.f || corr[1][0] != 1.f ||
+                                  corr[1][1] != 1.f)) {
 #pragma unroll
-  for (int mp = 0; mp < 2; ++mp)
+    for (int mp = 0; mp < 2; ++mp)
 #pragma unroll
-    for (int n = 0; n < DVT; ++n) {
-      o[mp][n][0] *= corr[mp][0]; o[mp][n][1] *= corr[mp][0];
-      o[mp][n][2] *= corr[mp][1]; o[mp][n][3] *= corr[mp][1];
-    }
+      for (int n = 0; n < DVT; ++n) {
+        o[mp][n][0] *= corr[mp][0]; o[mp][n][1] *= corr[mp][0];
+        o[mp][n][2] *= corr[mp][1]; o[mp][n][3] *= corr[mp][1];
+      }
+  }
 #pragma unroll
   for (int kk = 0; kk < KT / 16; ++kk) {
 #pragma unroll
@@ -213,11 +243,14 @@ __global__ void __launch_bounds__(DA_THREADS) diff_prefill_mma_kernel(
 #pragma unroll
     for (int n = 0; n < DVT; ++n) o[mp][n][0] = o[mp][n][1] = o[mp][n][2] = o[mp][n][3] = 0.f;
   }
+  const DaWalk walk_k = da_walk(2 * d, tid, DA_THREADS), walk_v = da_walk(dv, tid, DA_THREADS);
   auto issue = [&](int n) {               // where[n & 1] holds tile n's cache rows
-    da_load_rows(Ks + (size_t)(n & 1) * DA_KEYS * pitch_k, pitch_k, k_cache, where[n & 1],
-                 DA_KEYS, 2 * d, tid, DA_THREADS);
-    da_load_rows(Vs + (size_t)(n & 1) * DA_KEYS * pitch_v, pitch_v, v_cache, where[n & 1],
-                 DA_KEYS, dv, tid, DA_THREADS);
+    const int* list = where[n & 1];
+    auto at = [&](int r) { return list[r]; };
+    da_load_rows(Ks + (size_t)(n & 1) * DA_KEYS * pitch_k, pitch_k, k_cache, DA_KEYS, walk_k,
+                 (DA_KEYS * walk_k.chunks + DA_THREADS - 1) / DA_THREADS, at);
+    da_load_rows(Vs + (size_t)(n & 1) * DA_KEYS * pitch_v, pitch_v, v_cache, DA_KEYS, walk_v,
+                 (DA_KEYS * walk_v.chunks + DA_THREADS - 1) / DA_THREADS, at);
   };
   auto look_up = [&](int n) {
     if (tid < DA_KEYS)
@@ -307,6 +340,7 @@ __global__ void __launch_bounds__(DA_THREADS) diff_decode_mma_kernel(
     int page_size, int num_pages, int max_splits, float scale_log2, int* __restrict__ err,
     float temp_coef, int temp_every) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
+  __shared__ uint64_t bars[DA_THREADS / 32][DA_DSTAGES];
   bf_pdl_trigger();
   bf_pdl_wait();
   const int Gh = nh / nkv, hblocks = (Gh + 15) / 16;
@@ -319,9 +353,15 @@ __global__ void __launch_bounds__(DA_THREADS) diff_decode_mma_kernel(
   if ((int)blockIdx.x * 4 * DA_SHARE > p) return;
   const int pitch_k = 2 * d + 8, pitch_v = dv + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);       // [16][pitch_k]
-  const size_t per_warp = (size_t)2 * DA_DKEYS * (pitch_k + pitch_v);
-  __nv_bfloat16* Ks = Qs + (size_t)16 * pitch_k + warp * per_warp;      // [2][32][pitch_k]
-  __nv_bfloat16* Vs = Ks + (size_t)2 * DA_DKEYS * pitch_k;              // [2][32][pitch_v]
+  constexpr int KT = DA_DKEYS, ST = DA_DSTAGES;
+  const size_t per_warp = (size_t)ST * KT * (pitch_k + pitch_v);
+  __nv_bfloat16* Ks = Qs + (size_t)16 * pitch_k + warp * per_warp;      // [ST][16][pitch_k]
+  __nv_bfloat16* Vs = Ks + (size_t)ST * KT * pitch_k;                   // [ST][16][pitch_v]
+  uint64_t* full = bars[warp];
+  if (lane == 0) {
+    for (int x = 0; x < ST; ++x) bf_mbar_init(full + x, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
   const int chunks = 2 * d >> 3;
   for (int i = tid; i < 16 * chunks; i += DA_THREADS) {
     const int hr = i / chunks, c = (i - hr * chunks) << 3;
@@ -336,7 +376,7 @@ __global__ void __launch_bounds__(DA_THREADS) diff_decode_mma_kernel(
   const int first = share * DA_SHARE;
   if (first > p || share >= max_splits) return;          // (no barrier of the CTA follows)
   const int* table = tables + (size_t)seq_of_token[t] * table_stride;
-  const int n_tiles = (min(p, first + DA_SHARE - 1) - first) / DA_DKEYS + 1;
+  const int n_tiles = (min(p, first + DA_SHARE - 1) - first) / KT + 1;
   const float sc0 = scale_log2 * bf_query_temperature(p, temp_coef, temp_every);
   const float sc[2] = {sc0, sc0};
   float m[2][2], l[2][2], corr[2][2];
@@ -348,55 +388,50 @@ __global__ void __launch_bounds__(DA_THREADS) diff_decode_mma_kernel(
 #pragma unroll
     for (int n = 0; n < DVT; ++n) o[mp][n][0] = o[mp][n][1] = o[mp][n][2] = o[mp][n][3] = 0.f;
   }
-  // a lane looks a key row up; all four tiles' lookups are in flight together
-  int at[DA_SHARE / DA_DKEYS];
+  // a lane looks a key row up; all lookups of the share are in flight together
+  int at[DA_SHARE / 32];
 #pragma unroll
-  for (int n = 0; n < DA_SHARE / DA_DKEYS; ++n)
-    at[n] = da_cache_row(table, first + n * DA_DKEYS + lane, p + 1, nkv, g, page_size, num_pages,
-                         err);
-  auto issue = [&](int n) {
+  for (int n = 0; n < DA_SHARE / 32; ++n)
+    at[n] = da_cache_row(table, first + n * 32 + lane, p + 1, nkv, g, page_size, num_pages, err);
+  // keys beyond p (masked, but their values must be finite) take the row of the share's first
+  const int safe = max(__shfl_sync(0xffffffffu, at[0], 0), 0);
+  auto issue = [&](int n) {               // 16 lanes fetch a key row each, 16 a value row
     int mine = -1;
 #pragma unroll
-    for (int x = 0; x < DA_SHARE / DA_DKEYS; ++x)
-      if (x == n) mine = at[x];
-    __nv_bfloat16* kt = Ks + (size_t)(n & 1) * DA_DKEYS * pitch_k;
-    __nv_bfloat16* vt = Vs + (size_t)(n & 1) * DA_DKEYS * pitch_v;
-    const int kc = 2 * d >> 3, vc = dv >> 3;
-#pragma unroll 4
-    for (int i = lane; i < DA_DKEYS * kc; i += 32) {
-      const int row = i / kc, c = (i - row * kc) << 3;
-      const int e = __shfl_sync(0xffffffffu, mine, row);
-      cp_async16(kt + (size_t)row * pitch_k + c,
-                 e >= 0 ? k_cache + (size_t)e * 2 * d + c : k_cache, e >= 0 ? 16 : 0);
-    }
-#pragma unroll 4
-    for (int i = lane; i < DA_DKEYS * vc; i += 32) {
-      const int row = i / vc, c = (i - row * vc) << 3;
-      const int e = __shfl_sync(0xffffffffu, mine, row);
-      cp_async16(vt + (size_t)row * pitch_v + c,
-                 e >= 0 ? v_cache + (size_t)e * dv + c : v_cache, e >= 0 ? 16 : 0);
-    }
-  };
-  issue(0);
-  cp_async_commit();
-  for (int n = 0; n < n_tiles; ++n) {
-    if (n + 1 < n_tiles) issue(n + 1);
-    cp_async_commit();
-    cp_async_wait<1>();
+    for (int x = 0; x < DA_SHARE / 32; ++x)
+      if (x == n / 2) mine = at[x];
+    const int row = lane & 15, st = n % ST;
+    int e = __shfl_sync(0xffffffffu, mine, row + (n & 1) * 16);
+    if (e < 0) e = safe;
+    if (lane == 0) bf_mbar_expect_tx(full + st, (uint32_t)(KT * (2 * d + dv) * 2));
     __syncwarp();
-    const __nv_bfloat16* kt = Ks + (size_t)(n & 1) * DA_DKEYS * pitch_k;
-    const __nv_bfloat16* vt = Vs + (size_t)(n & 1) * DA_DKEYS * pitch_v;
-    const int last = p - (first + n * DA_DKEYS);
+    if (lane < 16)
+      bf_bulk_load(Ks + ((size_t)st * KT + row) * pitch_k, k_cache + (size_t)e * 2 * d,
+                   (uint32_t)(4 * d), full + st);
+    else
+      bf_bulk_load(Vs + ((size_t)st * KT + row) * pitch_v, v_cache + (size_t)e * dv,
+                   (uint32_t)(2 * dv), full + st);
+  };
+  for (int n = 0; n < min(ST, n_tiles); ++n) issue(n);
+  for (int n = 0; n < n_tiles; ++n) {
+    if (!bf_mbar_wait_bounded(full + n % ST, (n / ST) & 1)) {
+      atomicOr(err, BF_ERR_WAIT);
+      break;
+    }
+    __syncwarp();
+    const __nv_bfloat16* kt = Ks + (size_t)(n % ST) * KT * pitch_k;
+    const __nv_bfloat16* vt = Vs + (size_t)(n % ST) * KT * pitch_v;
+    const int last = p - (first + n * KT);
     const int rel[2] = {last, last};
-    uint32_t pa[2][DA_DKEYS / 16][4];
+    uint32_t pa[2][KT / 16][4];
 #pragma unroll
     for (int mp = 0; mp < 2; ++mp)
-      da_scores<DA_DKEYS>(Qs + mp * d, pitch_k, kt + mp * d, pitch_k, d, lane, rel,
-                          last >= DA_DKEYS - 1, sc, m[mp], l[mp], corr[mp], pa[mp]);
-    da_values<DA_DKEYS, DVT>(vt, pitch_v, dv, lane, pa, corr, o);
+      da_scores<KT>(Qs + mp * d, pitch_k, kt + mp * d, pitch_k, d, lane, rel,
+                    last >= KT - 1, sc, m[mp], l[mp], corr[mp], pa[mp]);
+    da_values<KT, DVT>(vt, pitch_v, dv, lane, pa, corr, o);
     __syncwarp();
+    if (n + ST < n_tiles) issue(n + ST);
   }
-  cp_async_wait<0>();
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int hr = (lane >> 2) + 8 * i;
@@ -477,7 +512,7 @@ BF_EXPORT int bf_diff_attention_decode_mma(
   dim3 grid((max_splits + 3) / 4, nkv * ((Gh + 15) / 16), n_rows);
   if (grid.y > 65535u || grid.z > 65535u) return (int)cudaErrorInvalidValue;
   const size_t smem =
-      (size_t)2 * (16 * (2 * d + 8) + 4 * 2 * DA_DKEYS * ((2 * d + 8) + (dv + 8)));
+      (size_t)2 * (16 * (2 * d + 8) + 4 * DA_DSTAGES * DA_DKEYS * ((2 * d + 8) + (dv + 8)));
   auto kern = dv <= 64 ? diff_decode_mma_kernel<8> : diff_decode_mma_kernel<16>;
   static bool configured[BF_MAX_DEVICES][2];
   bool& c = configured[bf_current_device()][dv <= 64 ? 0 : 1];

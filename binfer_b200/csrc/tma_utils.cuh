@@ -125,6 +125,15 @@ __device__ __forceinline__ void bf_tma_load_2d(void* smem_dst, const CUtensorMap
       "l"(map), "r"(bf_smem_u32(bar)), "r"(x), "r"(y)
       : "memory");
 }
+// Untiled bulk copy global -> shared; both addresses 16-byte aligned, bytes a multiple of 16.
+__device__ __forceinline__ void bf_bulk_load(void* smem_dst, const void* src, uint32_t bytes,
+                                             uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::
+          "r"(bf_smem_u32(smem_dst)),
+      "l"(src), "r"(bytes), "r"(bf_smem_u32(bar))
+      : "memory");
+}
 // A box from shared memory to the matrix, in this thread's current bulk group (x: column, a
 // multiple of 8 elements; no coordinate negative).
 __device__ __forceinline__ void bf_tma_store_2d(const CUtensorMap* map, const void* smem_src,

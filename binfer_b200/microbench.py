@@ -2,6 +2,8 @@
 
     python -m binfer_b200.microbench decode_attention --batch 8 --ctx 4096
     python -m binfer_b200.microbench prefill_attention --tokens 2048
+    python -m binfer_b200.microbench diff_prefill --tokens 2048 --head-dim 64 --value-dim 128
+    python -m binfer_b200.microbench diff_decode --batch 8 --head-dim 64 --value-dim 128
     python -m binfer_b200.microbench gemm --tokens 8 --features 6144 --k 4096 [--library]
     python -m binfer_b200.microbench add_rmsnorm --tokens 8 --hidden 4096
     BINFER_B200_TRACE=1 python -m binfer_b200.microbench step_timeline --batch 8 --ctx 4096 --layers 6
@@ -148,6 +150,53 @@ def prefill_attention(a):
     flops = 4.0 * nh * d * (T * start + T * (T + 1) / 2)
     report("prefill_attention", us, flops=flops, tokens=T, start=start, heads=nh, kv_heads=nkv,
            head_dim=d)
+
+
+def _diff_cache(dev, a, n_req, ctx, sets):
+    """Caches for differential attention: key rows of both maps side by side, 2 * head_dim."""
+    keys = _paged_cache(dev, n_req, ctx, a.kv_heads, 2 * a.head_dim, a.page_size, sets, a.scattered)
+    return [(kc, torch.randn(*kc.shape[:3], a.value_dim, device=dev, dtype=BF16), bt)
+            for kc, _, bt in keys]
+
+
+def diff_decode(a):
+    dev = torch.device("cuda:0")
+    B, ctx, nh, nkv, d, dv = a.batch, a.ctx, a.heads, a.kv_heads, a.head_dim, a.value_dim
+    per_set = B * ctx * nkv * (2 * d + dv) * 2
+    caches = _diff_cache(dev, a, B, ctx, max(2, int(3e8 // per_set) + 1))
+    q = torch.randn(B, nh * 2 * d, device=dev, dtype=BF16)
+    gate = torch.randn(B, nh * dv, device=dev, dtype=BF16)
+    out = torch.empty_like(gate)
+    dc = ops.DiffCombine(0.7, 1e-5, 0.5, gate, 0.1, 1024)
+    sot = torch.arange(B, dtype=torch.int32, device=dev)
+    pos = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+    err = ops.error_word(dev)
+    variant = a.variant if a.variant in ("persistent", "mma_sync") else "auto"
+    fns = [lambda c=c: ops.diff_attention_decode(q, c[0], c[1], None, B, sot, pos, c[2], out, nh,
+                                                 d ** -0.5, dc, ctx, err, variant=variant)
+           for c in caches]
+    us = timed(fns, a.iters, a.warmup)
+    report("diff_decode", us, nbytes=per_set, batch=B, ctx=ctx, heads=nh, kv_heads=nkv,
+           map_dim=d, value_dim=dv, page_size=a.page_size, variant=variant)
+
+
+def diff_prefill(a):
+    dev = torch.device("cuda:0")
+    T, start, nh, d, dv = a.tokens, a.start, a.heads, a.head_dim, a.value_dim
+    (kc, vc, bt), = _diff_cache(dev, a, 1, start + T, 1)
+    q = torch.randn(T, nh * 2 * d, device=dev, dtype=BF16)
+    gate = torch.randn(T, nh * dv, device=dev, dtype=BF16)
+    out = torch.empty_like(gate)
+    dc = ops.DiffCombine(0.7, 1e-5, 0.5, gate, 0.1, 1024)
+    items = torch.tensor([[0, 0, T, start]], dtype=torch.int32, device=dev)
+    err = ops.error_word(dev)
+    variant = a.variant if a.variant in ("umma", "mma_sync") else "auto"
+    fn = lambda: ops.diff_attention_prefill(q, kc, vc, items, 1, T, bt, out, nh, d ** -0.5, dc,
+                                            err, max_ctx=start + T, variant=variant)
+    us = timed([fn], a.iters, a.warmup)
+    flops = 2.0 * 2 * nh * (d + dv) * (T * start + T * (T + 1) / 2)
+    report("diff_prefill", us, flops=flops, tokens=T, start=start, heads=nh, kv_heads=a.kv_heads,
+           map_dim=d, value_dim=dv, variant=variant)
 
 
 def gemm(a):
@@ -335,7 +384,8 @@ def main(argv=None):
     ap = argparse.ArgumentParser(prog="python -m binfer_b200.microbench", description=__doc__,
                                  formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("kernel", choices=["decode_attention", "prefill_attention", "gemm",
-                                       "swiglu", "add_rmsnorm", "step_timeline", "scan"])
+                                       "swiglu", "add_rmsnorm", "step_timeline", "scan",
+                                       "diff_decode", "diff_prefill"])
     ap.add_argument("--iters", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--batch", type=int, default=8)
@@ -345,6 +395,8 @@ def main(argv=None):
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--head-dim", type=int, default=128)
+    ap.add_argument("--value-dim", type=int, default=128, help="diff_*: size of a value head "
+                                                              "(--head-dim: of one map's key)")
     ap.add_argument("--page-size", type=int, default=16)
     ap.add_argument("--scattered", action="store_true",
                     help="decode_attention: no two pages of a tile side by side in the pool")
@@ -379,7 +431,8 @@ def main(argv=None):
     GRAPH = not a.no_graph
     {"decode_attention": decode_attention, "prefill_attention": prefill_attention,
      "gemm": gemm, "swiglu": swiglu, "add_rmsnorm": add_rmsnorm,
-     "step_timeline": step_timeline, "scan": scan}[a.kernel](a)
+     "step_timeline": step_timeline, "scan": scan, "diff_decode": diff_decode,
+     "diff_prefill": diff_prefill}[a.kernel](a)
     return 0
 
 
