@@ -77,6 +77,8 @@ def _register_builtin() -> None:
     register_architecture("Folivik", FolivikConfig.from_dict)
     from .pabelix import PabelixConfig
     register_architecture("Pabelix", PabelixConfig.from_dict)
+    from .nazorax import NazoraxConfig
+    register_architecture("Nazorax", NazoraxConfig.from_dict)
 
 
 _register_builtin()

@@ -69,11 +69,15 @@ class NormSpec:
     """``offset``: what is added to the stored weight to get the one that multiplies (1.0 for
     a family whose norm weights hold the deviation from one)."""
 
-    kind: str = "rmsnorm"      # or "layernorm": mean taken off, weight and bias
+    kind: str = "rmsnorm"      # or "layernorm": mean taken off, weight and bias; or "tanh_norm":
+                               # tanh(alpha x) * weight + bias, no statistic of the row (no eps)
     eps: float = 1e-6
     offset: float = 0.0
-    # layernorm: what follows the weight tensor's name to give the bias tensor's (None: no bias)
+    # layernorm, tanh_norm: what follows the weight tensor's name to give the bias tensor's (None:
+    # no bias)
     bias_suffix: Optional[str] = None
+    # tanh_norm: the same for the tensor of one number, alpha
+    alpha_suffix: str = ".alpha"
     # rmsnorm: the weight tensor is a single number that multiplies every coordinate
     scalar_weight: bool = False
 
@@ -136,6 +140,8 @@ class GatedMLPSpec:
     up_offset: float = 0.0
     # the tensors' names inside the feed-forward's prefix: gate, up, down
     names: Tuple[str, str, str] = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+    # with ``bias``: the biases' names, in the same order
+    bias_names: Tuple[str, str, str] = ("gate_proj.bias", "up_proj.bias", "down_proj.bias")
 
 
 @dataclass(frozen=True)
@@ -218,7 +224,9 @@ class ConvWindowAttentionSpec:
     of ``head_dim`` numbers that the heads share (tensors ``q_head_norm``, ``k_head_norm``).
     ``head_temperature``: head h's scores are multiplied by the number ``temp[h]`` (a tensor of
     the mixer).  ``log_distance_bias``: ``b1_h ln(1 + b2_h (i - j))`` is taken off the score of
-    query i and key j (tensors ``bias_slope`` b1 and ``bias_rate`` b2, one number per head)."""
+    query i and key j (tensors ``bias_slope`` b1 and ``bias_rate`` b2, one number per head).
+    ``proj_bias``: the q, k and v projections have biases (the projection's name with
+    ``bias_suffix``; without a convolution only)."""
 
     kind: str = "conv_window_attention"
     num_heads: int = 0
@@ -244,6 +252,8 @@ class ConvWindowAttentionSpec:
                                           ("k_head_norm", "k.norm"), ("temp", "temp"),
                                           ("bias_slope", "r1"), ("bias_rate", "r2"))
     conv_suffix: str = ".conv"
+    proj_bias: bool = False
+    bias_suffix: str = ".b"
 
     @property
     def softmax_scale(self) -> float:
@@ -290,7 +300,9 @@ class LatentAttentionSpec:
     per head.  ``position``: the rotation of the ``rot_dim`` parts (layout and offset are
     set by the mixer).  ``q_rank`` > 0: the queries go through a latent too, ``q = W_uq
     rmsnorm(W_dq h)`` with a weight of ``q_rank`` numbers (tensors ``dq``, ``dq_norm``, ``uq``
-    in place of ``q``).  ``names``: the tensors inside the mixer's prefix."""
+    in place of ``q``).  ``sinks``: a learned logit per head (tensor ``sink``) joins the
+    softmax's denominator; it has no key and no value and is not scaled.  ``names``: the tensors
+    inside the mixer's prefix."""
 
     kind: str = "latent_attention"
     num_heads: int = 0
@@ -303,9 +315,11 @@ class LatentAttentionSpec:
     position: Optional[RopeSpec] = None
     head_gate: bool = True
     q_rank: int = 0
+    sinks: bool = False
     names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("dkv", "dkv"), ("dkv_norm", "dkv.norm"),
                                           ("uk", "uk"), ("uv", "uv"), ("g", "g"), ("o", "o"),
-                                          ("dq", "dq"), ("dq_norm", "dq.norm"), ("uq", "uq"))
+                                          ("dq", "dq"), ("dq_norm", "dq.norm"), ("uq", "uq"),
+                                          ("sink", "sink"))
 
     @property
     def softmax_scale(self) -> float:
@@ -449,7 +463,10 @@ class MoESpec:
     ``scoring`` "sigmoid": the scores are the sigmoids of the router outputs, each on its own;
     everything else as for "softmax_all".  ``group_top``: a group counts by the sum of its
     that many largest choice scores.  ``normalize`` False: the chosen scores are not divided
-    by their sum."""
+    by their sum.
+
+    ``activation`` "clamped": the experts are of the clamped form of :class:`GatedMLPSpec`, with
+    ``limit`` for the chosen ones and ``shared_limit`` for the shared one."""
 
     kind: str = "moe"
     num_experts: int = 0
@@ -473,6 +490,10 @@ class MoESpec:
     identity: int = 0
     group_top: int = 1
     normalize: bool = True
+    limit: float = 0.0           # "clamped" only, like the three below
+    shared_limit: float = 0.0
+    slope: float = 1.0
+    up_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -491,13 +512,16 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class PassStart:
-    """What is added to the residual stream right before a schedule entry that opens a pass
-    over a run of layers that is walked several times: the embedding output once more
-    (``embedding``), then row ``row`` of the model's table of pass vectors
-    (:attr:`ModelSpec.pass_table`; None: nothing)."""
+    """What happens to the residual stream right before a schedule entry that opens a pass
+    over a run of layers that is walked several times: it takes the embedding output once more
+    (``embedding``) and row ``row`` of the model's table of pass vectors
+    (:attr:`ModelSpec.pass_table`; None: nothing); or (``project``) it becomes the product of
+    the model's pass projection (:attr:`ModelSpec.pass_projection`) with itself and the embedding
+    output side by side, ``x <- W [x; x0]``."""
 
     embedding: bool = False
     row: Optional[int] = None
+    project: bool = False
 
 
 @dataclass(frozen=True)
@@ -544,6 +568,9 @@ class ModelSpec:
     # (tensor name, rows) of a table ``[rows, hidden_size]`` whose rows schedule entries add
     # to the stream (ScheduleEntry.before); None: the model has none
     pass_table: Optional[Tuple[str, int]] = None
+    # name of a matrix ``[hidden_size, 2 hidden_size]`` for schedule entries that project the
+    # stream and the embedding output (ScheduleEntry.before); None: the model has none
+    pass_projection: Optional[str] = None
     # added to the embedding output; None: nothing (positions enter in the mixers only)
     position_vectors: Optional[PositionVectorSpec] = None
 

@@ -19,7 +19,8 @@
 //   O += P V for every fourth pair of 8-column value tiles (pairs qt, qt + 4, ...).
 // Each row masks by its own token's position.  With `splits` > 1 (steps of single tokens) the
 // key tiles of a request are shared out over that many CTAs, whose maxima, sums and raw
-// outputs a second kernel makes one.
+// outputs a second kernel makes one.  `sinks` (a logit per head, or null) join the rows' sums at
+// the end: in this kernel, or in the one that merges the shares.
 //
 // Sizes: rank and dr multiples of 16, rank at most 512, W at most 640.
 #include "common.cuh"
@@ -34,6 +35,14 @@ __device__ __forceinline__ float lat_ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// 1 / (L + the head's sink) where L is a sum of 2^(s - m): a sink z adds 2^(z log2(e) - m).  A sink
+// far above the maximum makes that infinite and the result zero, which is its limit.
+__device__ __forceinline__ float lat_inverse(float L, float m, const float* __restrict__ sinks,
+                                             int h) {
+  if (sinks) L += exp2f(fmaf(sinks[h], 1.4426950408889634f, -m));
+  return L > 0.f ? 1.f / L : 0.f;
 }
 
 // Keys `first .. first + 63` of a request (through its block table) on their way into a
@@ -73,7 +82,8 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_attention_kernel(
     const int* __restrict__ q_start, const int* __restrict__ positions,
     const int* __restrict__ tables, int table_stride, __nv_bfloat16* __restrict__ out, int H,
     int W, int rank, int page_size, int num_pages, float scale_log2, float* __restrict__ part_o,
-    float* __restrict__ part_ml, int splits, int* __restrict__ err) {
+    float* __restrict__ part_ml, int splits, const float* __restrict__ sinks,
+    int* __restrict__ err) {
   extern __shared__ __align__(16) unsigned char lat_smem[];
   const int pitch = W + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(lat_smem);       // [32][pitch]
@@ -286,7 +296,7 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_attention_kernel(
   for (int i = 0; i < 2; ++i) {
     const int r = row0 + mt * 16 + (lane >> 2) + 8 * i;
     if (r >= rows_total) continue;
-    const float inv = L[i] > 0.f ? 1.f / L[i] : 0.f;
+    const float inv = lat_inverse(L[i], m[i], sinks, r % H);
     __nv_bfloat16* dst = out + ((size_t)t0 * H + r) * rank;
 #pragma unroll
     for (int np = 0; np < NP; ++np) {
@@ -306,7 +316,8 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_attention_kernel(
 __global__ void latent_merge_kernel(const float* __restrict__ part_o,
                                     const float* __restrict__ part_ml, int splits,
                                     const int* __restrict__ q_start,
-                                    __nv_bfloat16* __restrict__ out, int H, int rank) {
+                                    __nv_bfloat16* __restrict__ out, int H, int rank,
+                                    const float* __restrict__ sinks) {
   const int r = blockIdx.x, tile = blockIdx.y, b = blockIdx.z;
   const int t0 = q_start[b], rows_total = (q_start[b + 1] - t0) * H;
   const int row = tile * LAT_ROWS + r;
@@ -319,7 +330,7 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_o,
     const float* ml = part_ml + (at + (size_t)x * LAT_ROWS + r) * 2;
     Lsum += ml[1] * lat_ex2(ml[0] - M);
   }
-  const float inv = Lsum > 0.f ? 1.f / Lsum : 0.f;
+  const float inv = lat_inverse(Lsum, M, sinks, row % H);
   __nv_bfloat16* dst = out + ((size_t)t0 * H + row) * rank;
   for (int c = threadIdx.x; c < rank; c += blockDim.x) {
     float acc = 0.f;
@@ -338,7 +349,8 @@ BF_EXPORT int bf_latent_attention(const void* q, const void* cache, const int* q
                                   const int* positions, const int* tables, int table_stride,
                                   void* out, int B, int max_rows, int H, int W, int rank,
                                   int page_size, int num_pages, float scale, float* part_o,
-                                  float* part_ml, int splits, int* err, cudaStream_t stream) {
+                                  float* part_ml, int splits, const float* sinks, int* err,
+                                  cudaStream_t stream) {
   if (B <= 0 || max_rows <= 0) return 0;
   if (W % 16 || rank % 16 || rank <= 0 || rank > 512 || W < rank || W > 640 || !(scale > 0.f))
     return (int)cudaErrorInvalidValue;
@@ -365,7 +377,7 @@ BF_EXPORT int bf_latent_attention(const void* q, const void* cache, const int* q
     latent_attention_kernel<N><<<grid, LAT_THREADS, smem, stream>>>(                            \
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, q_start, positions, tables,       \
         table_stride, (__nv_bfloat16*)out, H, W, rank, page_size, num_pages, scale * log2e,     \
-        part_o, part_ml, splits, err);                                                          \
+        part_o, part_ml, splits, sinks, err);                                                   \
   }
   if (NP == 2) LAT_GO(2, 0) else if (NP == 4) LAT_GO(4, 1) else LAT_GO(8, 2)
 #undef LAT_GO
@@ -373,7 +385,7 @@ BF_EXPORT int bf_latent_attention(const void* q, const void* cache, const int* q
     const int e = bf_launch_status();
     if (e) return e;
     latent_merge_kernel<<<dim3(LAT_ROWS, tiles, B), 128, 0, stream>>>(
-        part_o, part_ml, splits, q_start, (__nv_bfloat16*)out, H, rank);
+        part_o, part_ml, splits, q_start, (__nv_bfloat16*)out, H, rank, sinks);
   }
   return bf_launch_status();
 }

@@ -8,7 +8,8 @@
 // in front has taken.  The cosines and sines are multiplied by `rot_mag`.  After the norm of the
 // heads q and k may be multiplied by a weight per size of a head that the heads share (`head_w`
 // [2][dk]: q's, then k's), and each q head by a number of its own (`q_head_scale` [nh]: a factor
-// on the head's scores).
+// on the head's scores).  Without a convolution the projections may have biases (`proj_bias`, one
+// number per channel), added first.
 //
 //   y_t[c] = sum_j w[c, j] * u_{t - taps + 1 + j}[c],   j = 0 .. taps-1
 //
@@ -64,7 +65,7 @@ __global__ void conv_encode_kernel(
     int T, int nh, int nkv, int dk, int dv, int page_size, long long num_slots, int unit_norm,
     float eps, int vec2, int hpw, int* __restrict__ err, const float* __restrict__ pre_factor,
     const float* __restrict__ pre_weight, const float* __restrict__ head_w,
-    const float* __restrict__ q_head_scale) {
+    const float* __restrict__ q_head_scale, const float* __restrict__ proj_bias) {
   extern __shared__ float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int heads_total = nh + 2 * nkv;
@@ -109,6 +110,10 @@ __global__ void conv_encode_kernel(
         }
       } else {
         y = ce_ld2(proj + (size_t)t * stride + c);
+        if (proj_bias) {
+          y.x += proj_bias[c];
+          y.y += proj_bias[c + 1];
+        }
       }
       buf[i] = y.x;
       buf[i + 1] = y.y;
@@ -128,6 +133,7 @@ __global__ void conv_encode_kernel(
         }
       } else {
         y = bf_ld(proj + (size_t)t * stride + c);
+        if (proj_bias) y += proj_bias[c];
       }
       buf[i] = y;
     }
@@ -188,11 +194,12 @@ BF_EXPORT int bf_conv_encode(
     int nh, int nkv, int dk, int dv, int page_size, long long num_slots, int unit_norm, float eps,
     int act_dtype, float* rope_table, int* err, const float* pre_factor,
     const float* pre_weight, float rot_mag, const float* head_w, const float* q_head_scale,
-    cudaStream_t stream) {
+    const float* proj_bias, cudaStream_t stream) {
   // rope_table: scratch, float [T][rot_half][2] (unused without a rotation)
   if (T <= 0) return 0;
   if (taps > CE_MAX_TAPS || (taps > 1 && !state)) return (int)cudaErrorInvalidValue;
   if (taps < 1) conv_w = nullptr;              // (one tap: a factor per channel, no state)
+  if (taps >= 1 && proj_bias) return (int)cudaErrorInvalidValue;
   if (!pre_factor || !pre_weight) pre_factor = pre_weight = nullptr;
   if (rot_half > 0) {
     if (!rope_table) return (int)cudaErrorInvalidValue;
@@ -220,14 +227,14 @@ BF_EXPORT int bf_conv_encode(
         (const float*)proj, stride, conv_w, taps, state, state_stride, state_slots, n_state_slots,
         seq_of_token, q_start, (const float2*)rope_table, rot_half, slots, (float*)q_out,
         q_stride, (float*)k_cache, (float*)v_cache, T, nh, nkv, dk, dv, page_size, num_slots,
-        unit_norm, eps, vec2, hpw, err, pre_factor, pre_weight, head_w, q_head_scale);
+        unit_norm, eps, vec2, hpw, err, pre_factor, pre_weight, head_w, q_head_scale, proj_bias);
   else
     conv_encode_kernel<__nv_bfloat16><<<blocks, warps * 32, smem, stream>>>(
         (const __nv_bfloat16*)proj, stride, conv_w, taps, state, state_stride, state_slots,
         n_state_slots, seq_of_token, q_start, (const float2*)rope_table, rot_half, slots,
         (__nv_bfloat16*)q_out, q_stride, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, T, nh,
         nkv, dk, dv, page_size, num_slots, unit_norm, eps, vec2, hpw, err, pre_factor,
-        pre_weight, head_w, q_head_scale);
+        pre_weight, head_w, q_head_scale, proj_bias);
   return bf_launch_status();
 }
 

@@ -208,26 +208,49 @@ BF_EXPORT int bf_add_rmsnorm(float* resid, const void* delta, const float* w, vo
 
 // --------------------------------------------------------------- residual add
 // resid[t, :] += delta[t, :]   (used when an add cannot ride on a following norm)
+// With `bias` (one number per column of rows of H) resid[t, c] += bias[c] as well.
 template <typename A>
 __global__ void residual_add_kernel(float* __restrict__ resid, const A* __restrict__ delta,
-                                    size_t n) {
+                                    size_t n, const float* __restrict__ bias, int H) {
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
-  for (; i < n; i += step) resid[i] += bf_ld(delta + i);
+  for (; i < n; i += step) resid[i] += bias ? bf_ld(delta + i) + bias[i % H] : bf_ld(delta + i);
+}
+
+// y[t, c] += bias[c] in the activation type: the bias of a product whose consumer takes none.
+template <typename A>
+__global__ void bias_add_kernel(A* __restrict__ y, size_t n, const float* __restrict__ bias, int H) {
+  size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const size_t step = (size_t)gridDim.x * blockDim.x;
+  for (; i < n; i += step) bf_st(y + i, bf_ld(y + i) + bias[i % H]);
+}
+
+BF_EXPORT int bf_bias_add(void* y, long long n, const float* bias, int H, int act_dtype,
+                          cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const int threads = 256;
+  long long blocks = (n + threads - 1) / threads;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (act_dtype == BF_DTYPE_F32)
+    bias_add_kernel<float><<<(int)blocks, threads, 0, stream>>>((float*)y, (size_t)n, bias, H);
+  else
+    bias_add_kernel<__nv_bfloat16><<<(int)blocks, threads, 0, stream>>>((__nv_bfloat16*)y,
+                                                                        (size_t)n, bias, H);
+  return bf_launch_status();
 }
 
 BF_EXPORT int bf_residual_add(float* resid, const void* delta, long long n, int act_dtype,
-                              cudaStream_t stream) {
+                              const float* bias, int H, cudaStream_t stream) {
   if (n <= 0) return 0;
   const int threads = 256;
   long long blocks = (n + threads - 1) / threads;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (act_dtype == BF_DTYPE_F32)
     residual_add_kernel<float><<<(int)blocks, threads, 0, stream>>>(resid, (const float*)delta,
-                                                                    (size_t)n);
+                                                                    (size_t)n, bias, H);
   else
     residual_add_kernel<__nv_bfloat16><<<(int)blocks, threads, 0, stream>>>(
-        resid, (const __nv_bfloat16*)delta, (size_t)n);
+        resid, (const __nv_bfloat16*)delta, (size_t)n, bias, H);
   return bf_launch_status();
 }
 
@@ -235,17 +258,21 @@ BF_EXPORT int bf_residual_add(float* resid, const void* delta, long long n, int 
 // out[t, c] = silu(gu[t, c]) * gu[t, I + c],  silu(g) = g / (1 + exp(-g))
 // (cuda/kernels/bf16_kernels.cu:461-477; there gate and up are separate buffers,
 // here they are the two halves of one fused projection's output row).
-// ACT: the activations of gate_act.cuh.
+// ACT: the activations of gate_act.cuh.  `bias` (2 I numbers, or null) is added to the row first.
 template <typename A, int ACT>
 __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, int T, int I,
-                                BfGateConst gk) {
+                                BfGateConst gk, const float* __restrict__ bias) {
   const size_t n = (size_t)T * I;
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
   for (; i < n; i += step) {
     const size_t t = i / I, c = i - t * I;
-    const float g = bf_ld(gu + t * 2 * I + c);
-    const float u = bf_ld(gu + t * 2 * I + I + c);
+    float g = bf_ld(gu + t * 2 * I + c);
+    float u = bf_ld(gu + t * 2 * I + I + c);
+    if (bias) {
+      g += bias[c];
+      u += bias[I + c];
+    }
     bf_st(out + i, bf_gate_mul<ACT>(g, u, gk));
   }
 }
@@ -302,7 +329,7 @@ __global__ void silu_mul_bf16_scaled_kernel(const __nv_bfloat16* __restrict__ gu
 template <int ACT>
 __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
                                          __nv_bfloat16* __restrict__ out, int T, int I,
-                                         BfGateConst gk) {
+                                         BfGateConst gk, const float* __restrict__ bias) {
   BF_TRACE_POINT(10 * BF_TR_SILU);
   bf_pdl_trigger();
   bf_pdl_wait();
@@ -331,7 +358,13 @@ __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
       __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o4);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
+        float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
+        if (bias) {
+          const float* bp = bias + (k ? c2 : c) + 2 * j;
+          const float2 bg = *reinterpret_cast<const float2*>(bp);
+          const float2 bu = *reinterpret_cast<const float2*>(bp + I);
+          g.x += bg.x; g.y += bg.y; u.x += bu.x; u.y += bu.y;
+        }
         o2[j] = __floats2bfloat162_rn(bf_gate_mul_fast<ACT>(g.x, u.x, gk),
                                       bf_gate_mul_fast<ACT>(g.y, u.y, gk));
       }
@@ -359,24 +392,25 @@ BF_EXPORT int bf_silu_mul_scaled(const void* gu, void* out, int T, int I,
 
 template <int ACT>
 static int gated_act_mul_launch(const void* gu, void* out, int T, int I, int act_dtype,
-                                cudaStream_t stream, BfGateConst gk = BfGateConst()) {
+                                cudaStream_t stream, BfGateConst gk = BfGateConst(),
+                                const float* bias = nullptr) {
   if (T <= 0) return 0;
   const int threads = 256;
   if (act_dtype == BF_DTYPE_BF16 && I % 8 == 0 && ((uintptr_t)gu & 15) == 0 &&
-      ((uintptr_t)out & 15) == 0) {
+      ((uintptr_t)out & 15) == 0 && ((uintptr_t)bias & 7) == 0) {
     long long blocks = ((long long)T * (I / 8) + threads - 1) / threads;
     if (blocks > 148 * 16) blocks = 148 * 16;
     return bf_launch_pdl(silu_mul_bf16_vec_kernel<ACT>, dim3((int)blocks), dim3(threads), 0,
-                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk);
+                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk, bias);
   }
   long long blocks = ((long long)T * I + threads - 1) / threads;
   if (blocks > 148 * 32) blocks = 148 * 32;
   if (act_dtype == BF_DTYPE_F32)
     silu_mul_kernel<float, ACT><<<(int)blocks, threads, 0, stream>>>((const float*)gu,
-                                                                    (float*)out, T, I, gk);
+                                                                    (float*)out, T, I, gk, bias);
   else
     silu_mul_kernel<__nv_bfloat16, ACT><<<(int)blocks, threads, 0, stream>>>(
-        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk);
+        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk, bias);
   return bf_launch_status();
 }
 
@@ -386,15 +420,17 @@ BF_EXPORT int bf_silu_mul(const void* gu, void* out, int T, int I, int act_dtype
 }
 
 // out[t, c] = act(gu[t, c]) * gu[t, I + c] with act 0: silu, 1: gelu's tanh form; 2: the clamped
-// form with its three constants (see BF_ACT_CLAMPED).
+// form with its three constants (see BF_ACT_CLAMPED); bias: null, or 2 I numbers added to gu first.
 BF_EXPORT int bf_gated_act_mul(const void* gu, void* out, int T, int I, int act, int act_dtype,
-                               float limit, float slope, float up_offset, cudaStream_t stream) {
+                               float limit, float slope, float up_offset, const float* bias,
+                               cudaStream_t stream) {
+  const BfGateConst gk = {limit, slope, up_offset};
   if (act == BF_ACT_CLAMPED)
-    return gated_act_mul_launch<BF_ACT_CLAMPED>(gu, out, T, I, act_dtype, stream,
-                                                BfGateConst{limit, slope, up_offset});
-  if (act == BF_ACT_SILU) return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream);
+    return gated_act_mul_launch<BF_ACT_CLAMPED>(gu, out, T, I, act_dtype, stream, gk, bias);
+  if (act == BF_ACT_SILU)
+    return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream, gk, bias);
   if (act == BF_ACT_GELU_TANH)
-    return gated_act_mul_launch<BF_ACT_GELU_TANH>(gu, out, T, I, act_dtype, stream);
+    return gated_act_mul_launch<BF_ACT_GELU_TANH>(gu, out, T, I, act_dtype, stream, gk, bias);
   return (int)cudaErrorInvalidValue;
 }
 

@@ -94,6 +94,7 @@ struct ClusterGemmParams {
   long long ldact;
   int inter;
   BfGateConst gk;
+  const float* gate_bias;       // [2 inter], added to f g and f u before the activation; or null
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -385,11 +386,24 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
         const int o0 = tile * h + c0;                     // first output of the chunk
         uint32_t packed[8];
 #pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          g[j] = __float_as_uint(__uint_as_float(g[j]) * factor);
+          u[j] = __float_as_uint(__uint_as_float(u[j]) * factor);
+        }
+        if (p.gate_bias) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c0 + j < h && o0 + j < p.inter) {
+              g[j] = __float_as_uint(__uint_as_float(g[j]) + __ldg(p.gate_bias + o0 + j));
+              u[j] = __float_as_uint(__uint_as_float(u[j]) + __ldg(p.gate_bias + p.inter + o0 + j));
+            }
+        }
+#pragma unroll
         for (int j = 0; j < 8; ++j) {
-          const float a = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j]) * factor,
-                                                  __uint_as_float(u[2 * j]) * factor, p.gk);
-          const float b = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j + 1]) * factor,
-                                                  __uint_as_float(u[2 * j + 1]) * factor, p.gk);
+          const float a = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j]),
+                                                  __uint_as_float(u[2 * j]), p.gk);
+          const float b = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j + 1]),
+                                                  __uint_as_float(u[2 * j + 1]), p.gk);
           packed[j] = pack_bf16x2(__float_as_uint(a), __float_as_uint(b));
         }
         __nv_bfloat16* dst = p.act_out + (size_t)row * p.ldact + o0;
@@ -940,13 +954,14 @@ BF_EXPORT int bf_gemm_swiglu_plan(int inter, int K, int num_sms, int* bn_out) {
 // rows first) and f the factor of the norm before the projection (row_partials as in
 // bf_silu_mul_scaled; null: 1), as one kernel for at most 64 token rows.  bn from
 // bf_gemm_swiglu_plan.  act_kind BF_ACT_CLAMPED: the clamped activation with its three constants
-// in silu's place.  Returns cudaErrorInvalidValue for what it does not take.
+// in silu's place.  gate_bias: null, or 2 inter floats added to f g and f u.  Returns
+// cudaErrorInvalidValue for what it does not take.
 BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int inter, int K,
                                   long long ldx, long long ldw, int bn, void* act,
                                   long long ldact, const float* row_partials, int row_count,
                                   int row_width, float row_eps, int* err, int act_kind,
                                   float limit, float slope, float up_offset,
-                                  cudaStream_t stream) {
+                                  const float* gate_bias, cudaStream_t stream) {
   if (tokens <= 0 || inter <= 0) return 0;
   if (act_kind != BF_ACT_SILU && act_kind != BF_ACT_CLAMPED) return (int)cudaErrorInvalidValue;
   if (tokens > CL_MAX_TOKENS || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) ||
@@ -963,6 +978,7 @@ BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int 
   p.act_out = (__nv_bfloat16*)act;
   p.ldact = ldact;
   p.inter = inter;
+  p.gate_bias = gate_bias;
   p.rs.partials = row_partials;
   p.rs.count = row_count;
   p.rs.inv_width = row_width > 0 ? 1.f / (float)row_width : 0.f;

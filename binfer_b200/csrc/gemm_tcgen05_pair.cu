@@ -49,6 +49,7 @@ struct PairParams {
   long long ldo;               // row stride of the output, in elements
   int* err;
   BfGateConst gk;          // of the clamped activation (gated 2)
+  const float* gate_bias;  // gated: [2 features], added to the sums before the activation; or null
 };
 
 constexpr int PM = 256;                      // token rows per tile (128 per CTA)
@@ -113,6 +114,20 @@ __device__ __forceinline__ void pair_arrive_remote(uint32_t bar_cluster_addr) {
 __device__ __forceinline__ float pair_gate(float g, float u, int gated, const BfGateConst& gk) {
   return gated == 2 ? bf_gate_mul_fast<BF_ACT_CLAMPED>(g, u, gk)
                     : bf_gate_mul_fast<BF_ACT_SILU>(g, u, gk);
+}
+
+// ... of N neighbouring outputs from o0 on, the biases added first (places beyond `features` stay
+// as they are: they are not stored)
+template <int N>
+__device__ __forceinline__ void pair_gate_bias(uint32_t (&g)[N], uint32_t (&u)[N], int o0,
+                                               const PairParams& p) {
+  if (!p.gate_bias) return;
+#pragma unroll
+  for (int j = 0; j < N; ++j)
+    if (o0 + j < p.features) {
+      g[j] = __float_as_uint(__uint_as_float(g[j]) + __ldg(p.gate_bias + o0 + j));
+      u[j] = __float_as_uint(__uint_as_float(u[j]) + __ldg(p.gate_bias + p.features + o0 + j));
+    }
 }
 
 template <typename OutT>
@@ -325,6 +340,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
                 const int col = slab * 128 + hs * 32;
                 tmem_ld32(taddr + col, r);
                 tmem_ld32(taddr + col + 64, up);
+                pair_gate_bias<32>(r, up, tf * 128 + slab * 64 + hs * 32, p);
 #pragma unroll
                 for (int j = 0; j < 32; ++j)
                   r[j] = __float_as_uint(pair_gate(__uint_as_float(r[j]), __uint_as_float(up[j]),
@@ -381,6 +397,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
               tmem_ld16_pair(taddr + half * 2 * q + c0, taddr + half * 2 * q + q + c0, g, up);
               const int o0 = tf * (p.bn >> 1) + half * q + c0;
               if (t < p.tokens && o0 < p.features) {
+                pair_gate_bias<16>(g, up, o0, p);
 #pragma unroll
                 for (int j = 0; j < 16; ++j)
                   g[j] = __float_as_uint(pair_gate(__uint_as_float(g[j]), __uint_as_float(up[j]),
@@ -524,14 +541,16 @@ BF_EXPORT int bf_gemm_pair_choose_bn(int tokens, int columns, int step, int num_
 // out[tokens, features] = x[tokens, K] * w[features, K]^T in bf16 with float accumulation, on
 // pairs of CTAs.  gated != 0: w is [2 features, K] (gate rows first) and out[t, o] =
 // silu(x . w[o]) * (x . w[features + o]), bf16 only; gated == 2: the clamped activation of
-// gate_act.cuh with its three constants instead.  out_dtype: BF_DTYPE_BF16 or
+// gate_act.cuh with its three constants instead; gate_bias ([2 features] floats, or null) is added
+// before the activation.  out_dtype: BF_DTYPE_BF16 or
 // BF_DTYPE_F32.  accumulate != 0 (float out only): out += the product.  bn: accumulator
 // columns per tile (0: chosen here).  Returns
 // cudaErrorInvalidValue for shapes it does not take.
 BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tokens, int features,
                                 int K, long long ldx, long long ldw, long long ldo, int out_dtype,
                                 int gated, int accumulate, int bn, int num_sms, int* err,
-                                float limit, float slope, float up_offset, cudaStream_t stream) {
+                                float limit, float slope, float up_offset,
+                                const float* gate_bias, cudaStream_t stream) {
   if (tokens <= 0 || features <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || num_sms < 2)
     return (int)cudaErrorInvalidValue;
@@ -550,6 +569,7 @@ BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tok
   p.bn = bn;
   p.gated = gated == 2 ? 2 : (gated ? 1 : 0);
   p.gk = BfGateConst{limit, slope, up_offset};
+  p.gate_bias = gated ? gate_bias : nullptr;
   p.accumulate = accumulate ? 1 : 0;
   p.tiles_t = (tokens + PM - 1) / PM;
   p.tiles_f = (columns + bn - 1) / bn;

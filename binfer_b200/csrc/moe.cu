@@ -23,11 +23,14 @@
 // moe_act: for experts whose gate and up projections are stacked into one product
 // `gu [T, 2F]` (gate rows of all experts, then up rows; F = E ff + ff_shared), the
 // activations of every expert scaled by the token's weight for that expert,
-//   act[t, c] = silu(gu[t, c]) * gu[t, F + c] * route_w[t, expert(c)],
-// so that one product with the stacked down projections gives the weighted sum.
+//   act[t, c] = A(gu[t, c], gu[t, F + c]) * route_w[t, expert(c)],
+// so that one product with the stacked down projections gives the weighted sum.  A is
+// silu(gate) up, or the clamped form with its constants (gate_act.cuh), of which the shared expert
+// has a set of its own.
 #include <float.h>
 
 #include "common.cuh"
+#include "gate_act.cuh"
 
 // One block per MR_TOKENS tokens: their rows go to shared memory as float; every warp takes a
 // slice of the width and, row by row of the router, its share of each token's dot product
@@ -299,10 +302,10 @@ BF_EXPORT int bf_moe_route(const void* h, long long stride, const float* w, int 
   return bf_launch_status();
 }
 
-template <typename A>
+template <typename A, int ACT>
 __global__ void moe_act_kernel(const A* __restrict__ gu, const float* __restrict__ route_w,
                                A* __restrict__ act, int T, int F, int E, int ff, int rw_cols,
-                               int shared_gate) {
+                               int shared_gate, BfGateConst gk, BfGateConst gk_sh) {
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (long long)T * F) return;
   const int t = (int)(i / F), c = (int)(i % F);
@@ -311,17 +314,19 @@ __global__ void moe_act_kernel(const A* __restrict__ gu, const float* __restrict
   float r = 0.f;
   if (wgt != 0.f) {
     const float g = bf_ld(gu + (size_t)t * 2 * F + c), u = bf_ld(gu + (size_t)t * 2 * F + F + c);
-    r = g / (1.f + expf(-g)) * u * wgt;
+    r = bf_gate_mul<ACT>(g, u, e < E ? gk : gk_sh) * wgt;
   }
   bf_st(act + i, r);
 }
 
 // bfloat16 with F, ff and the experts' total a multiple of 8: eight columns a thread (they
 // belong to one expert), 16-byte loads and stores.
+template <int ACT>
 __global__ void moe_act_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
                                         const float* __restrict__ route_w,
                                         __nv_bfloat16* __restrict__ act, int T, int F, int E,
-                                        int ff, int rw_cols, int shared_gate) {
+                                        int ff, int rw_cols, int shared_gate, BfGateConst gk,
+                                        BfGateConst gk_sh) {
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   const int F8 = F >> 3;
   if (i >= (long long)T * F8) return;
@@ -335,39 +340,57 @@ __global__ void moe_act_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
     const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
     const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&u4);
     __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+    const BfGateConst k = e < E ? gk : gk_sh;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
-      o2[j] = __floats2bfloat162_rn(g.x / (1.f + expf(-g.x)) * u.x * wgt,
-                                    g.y / (1.f + expf(-g.y)) * u.y * wgt);
+      o2[j] = __floats2bfloat162_rn(bf_gate_mul<ACT>(g.x, u.x, k) * wgt,
+                                    bf_gate_mul<ACT>(g.y, u.y, k) * wgt);
     }
   }
   *reinterpret_cast<uint4*>(act + (size_t)t * F + c) = out;
 }
 
 // rw_cols: the columns of a row of route_w; shared_gate: column E holds the shared expert's
-// weight (else that expert's weight is one)
-BF_EXPORT int bf_moe_act(const void* gu, const float* route_w, void* act, int T, int F, int E,
-                         int ff, int rw_cols, int shared_gate, int act_dtype,
-                         cudaStream_t stream) {
-  if (T <= 0 || F <= 0) return 0;
+// weight (else that expert's weight is one).  act_kind: BF_ACT_SILU, or BF_ACT_CLAMPED with its
+// constants (the shared expert's limit apart)
+template <int ACT>
+static int moe_act_launch(const void* gu, const float* route_w, void* act, int T, int F, int E,
+                          int ff, int rw_cols, int shared_gate, int act_dtype, BfGateConst gk,
+                          BfGateConst gk_sh, cudaStream_t stream) {
   const long long n = (long long)T * F;
   const unsigned blocks = (unsigned)((n + 255) / 256);
   if (act_dtype == BF_DTYPE_BF16 && F % 8 == 0 && ff % 8 == 0 &&
       (((uintptr_t)gu | (uintptr_t)act) & 15) == 0) {
-    moe_act_bf16_vec_kernel<<<(unsigned)((n / 8 + 255) / 256), 256, 0, stream>>>(
+    moe_act_bf16_vec_kernel<ACT><<<(unsigned)((n / 8 + 255) / 256), 256, 0, stream>>>(
         (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, T, F, E, ff, rw_cols,
-        shared_gate);
+        shared_gate, gk, gk_sh);
     return bf_launch_status();
   }
   if (act_dtype == BF_DTYPE_F32)
-    moe_act_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, route_w, (float*)act, T,
-                                                      F, E, ff, rw_cols, shared_gate);
+    moe_act_kernel<float, ACT><<<blocks, 256, 0, stream>>>((const float*)gu, route_w, (float*)act,
+                                                           T, F, E, ff, rw_cols, shared_gate, gk,
+                                                           gk_sh);
   else
-    moe_act_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(
+    moe_act_kernel<__nv_bfloat16, ACT><<<blocks, 256, 0, stream>>>(
         (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, T, F, E, ff, rw_cols,
-        shared_gate);
+        shared_gate, gk, gk_sh);
   return bf_launch_status();
+}
+
+BF_EXPORT int bf_moe_act(const void* gu, const float* route_w, void* act, int T, int F, int E,
+                         int ff, int rw_cols, int shared_gate, int act_dtype, int act_kind,
+                         float limit, float shared_limit, float slope, float up_offset,
+                         cudaStream_t stream) {
+  if (T <= 0 || F <= 0) return 0;
+  const BfGateConst gk = {limit, slope, up_offset}, gk_sh = {shared_limit, slope, up_offset};
+  if (act_kind == BF_ACT_CLAMPED)
+    return moe_act_launch<BF_ACT_CLAMPED>(gu, route_w, act, T, F, E, ff, rw_cols, shared_gate,
+                                          act_dtype, gk, gk_sh, stream);
+  if (act_kind == BF_ACT_SILU)
+    return moe_act_launch<BF_ACT_SILU>(gu, route_w, act, T, F, E, ff, rw_cols, shared_gate,
+                                       act_dtype, gk, gk_sh, stream);
+  return (int)cudaErrorInvalidValue;
 }
 
 // out[t, c] += h[t, c] * route_w[t, col]: the experts that return their input.
@@ -515,14 +538,15 @@ __device__ __forceinline__ void ms_dots(const A* __restrict__ w, size_t row_stri
 }
 
 // grid (row tiles, choices, T)
-template <typename A>
+template <typename A, int ACT>
 __global__ void moe_sparse_gate_up_kernel(const A* __restrict__ h, long long stride,
                                           const A* __restrict__ w_gu, int width, int F, int E,
                                           int ff, int ff_sh, int top,
                                           const int* __restrict__ top_ids,
                                           const float* __restrict__ top_w,
                                           const float* __restrict__ route_w, int rw_cols,
-                                          int shared_gate, A* __restrict__ act) {
+                                          int shared_gate, A* __restrict__ act,
+                                          BfGateConst gk, BfGateConst gk_sh) {
   extern __shared__ __align__(16) float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.z, k = blockIdx.y;
@@ -550,7 +574,8 @@ __global__ void moe_sparse_gate_up_kernel(const A* __restrict__ h, long long str
   ms_dots<A, MS_ROWS>(w_gu + ((size_t)F + base + row0) * width, (size_t)width, rows, sh, width,
                       lane, vec, u);
   if (lane == 0)
-    for (int r = 0; r < rows; ++r) bf_st(dst + row0 + r, g[r] / (1.f + expf(-g[r])) * u[r] * wgt);
+    for (int r = 0; r < rows; ++r)
+      bf_st(dst + row0 + r, bf_gate_mul<ACT>(g[r], u[r], shared ? gk_sh : gk) * wgt);
 }
 
 // grid (row tiles, T)
@@ -601,8 +626,11 @@ BF_EXPORT int bf_moe_sparse(const void* h, long long stride, const void* w_gu, c
                             const int* top_ids, const float* top_w, const float* route_w,
                             int rw_cols, void* act, void* out, int T, int width, int E, int ff,
                             int ff_sh, int top, int act_dtype, int shared_gate, int id_col,
-                            cudaStream_t stream) {
+                            int act_kind, float limit, float shared_limit, float slope,
+                            float up_offset, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (act_kind != BF_ACT_SILU && act_kind != BF_ACT_CLAMPED) return (int)cudaErrorInvalidValue;
+  const BfGateConst gk = {limit, slope, up_offset}, gk_sh = {shared_limit, slope, up_offset};
   const int F = E * ff + ff_sh;
   const int choices = top + (ff_sh ? 1 : 0);
   const int n_act = top * ff + ff_sh;
@@ -613,16 +641,20 @@ BF_EXPORT int bf_moe_sparse(const void* h, long long stride, const void* w_gu, c
   dim3 g1((rows_max + per_block - 1) / per_block, choices, T);
   dim3 g2((width + per_block - 1) / per_block, T);
   if (act_dtype == BF_DTYPE_F32) {
-    moe_sparse_gate_up_kernel<float><<<g1, MS_WARPS * 32, (size_t)width * 4, stream>>>(
+    auto k1 = act_kind == BF_ACT_CLAMPED ? moe_sparse_gate_up_kernel<float, BF_ACT_CLAMPED>
+                                         : moe_sparse_gate_up_kernel<float, BF_ACT_SILU>;
+    k1<<<g1, MS_WARPS * 32, (size_t)width * 4, stream>>>(
         (const float*)h, stride, (const float*)w_gu, width, F, E, ff, ff_sh, top, top_ids, top_w,
-        route_w, rw_cols, shared_gate, (float*)act);
+        route_w, rw_cols, shared_gate, (float*)act, gk, gk_sh);
     moe_sparse_down_kernel<float><<<g2, MS_WARPS * 32, (size_t)n_act * 4, stream>>>(
         (const float*)act, (const float*)w_down, width, F, E, ff, ff_sh, top, top_ids,
         (float*)out, (const float*)h, stride, route_w, rw_cols, id_col);
   } else {
-    moe_sparse_gate_up_kernel<__nv_bfloat16><<<g1, MS_WARPS * 32, (size_t)width * 4, stream>>>(
+    auto k1 = act_kind == BF_ACT_CLAMPED ? moe_sparse_gate_up_kernel<__nv_bfloat16, BF_ACT_CLAMPED>
+                                         : moe_sparse_gate_up_kernel<__nv_bfloat16, BF_ACT_SILU>;
+    k1<<<g1, MS_WARPS * 32, (size_t)width * 4, stream>>>(
         (const __nv_bfloat16*)h, stride, (const __nv_bfloat16*)w_gu, width, F, E, ff, ff_sh, top,
-        top_ids, top_w, route_w, rw_cols, shared_gate, (__nv_bfloat16*)act);
+        top_ids, top_w, route_w, rw_cols, shared_gate, (__nv_bfloat16*)act, gk, gk_sh);
     moe_sparse_down_kernel<__nv_bfloat16><<<g2, MS_WARPS * 32, (size_t)n_act * 4, stream>>>(
         (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, width, F, E, ff, ff_sh, top,
         top_ids, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, stride, route_w, rw_cols, id_col);

@@ -141,10 +141,74 @@ def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torc
                                 _c_int(1 if write_back else 0), _stream())
 
 
-def residual_add(resid: torch.Tensor, delta: torch.Tensor) -> None:
+def residual_add(resid: torch.Tensor, delta: torch.Tensor,
+                 bias: Optional[torch.Tensor] = None) -> None:
+    """resid[t] += delta[t] (+ bias)."""
     _want(resid, torch.float32, "resid")
+    if bias is not None:
+        _want(bias, torch.float32, "bias")
+        if bias.numel() != resid.shape[-1]:
+            raise KernelError("residual_add: bias must have the stream's width")
     _run("residual_add", lib().bf_residual_add, _ptr(resid), _ptr(delta), _c_ll(resid.numel()),
-                                 _c_int(_dtype_code(delta)), _stream())
+         _c_int(_dtype_code(delta)), _ptr(bias), _c_int(resid.shape[-1]), _stream())
+
+
+def bias_add(y: torch.Tensor, bias: torch.Tensor) -> None:
+    """y[t] += bias, in y's own type."""
+    _want(bias, torch.float32, "bias")
+    if not y.is_contiguous() or bias.numel() != y.shape[-1]:
+        raise KernelError("bias_add: y must be contiguous and as wide as the bias")
+    _run("bias_add", lib().bf_bias_add, _ptr(y), _c_ll(y.numel()), _ptr(bias),
+         _c_int(y.shape[-1]), _c_int(_dtype_code(y)), _stream())
+
+
+def _stream_deltas(what: str, resid, deltas, bias, act: torch.dtype) -> None:
+    _want(resid, torch.float32, "resid")
+    for d in deltas:
+        if d is not None and (d.dtype != act or not d.is_contiguous() or d.shape != resid.shape):
+            raise KernelError(f"{what}: a delta must be contiguous, of the stream's shape and of "
+                              f"the activation type")
+    if bias is not None:
+        _want(bias, torch.float32, "bias")
+        if bias.numel() != resid.shape[1]:
+            raise KernelError(f"{what}: bias must have the stream's width")
+
+
+def add_tanh_norm(resid: torch.Tensor, delta: Optional[torch.Tensor],
+                  delta2: Optional[torch.Tensor], bias: Optional[torch.Tensor], alpha: float,
+                  weight: torch.Tensor, shift: Optional[torch.Tensor], out: torch.Tensor,
+                  rows: Optional[torch.Tensor] = None, write_back: bool = True) -> None:
+    """out[i] = tanh(alpha (resid[r] + delta[r] + delta2[r] + bias)) * weight + shift with r =
+    rows[i] (or i); the sum is written back to resid when ``write_back``."""
+    _stream_deltas("add_tanh_norm", resid, (delta, delta2), bias, out.dtype)
+    _want(weight, torch.float32, "weight")
+    n, H = out.shape
+    if shift is not None:
+        _want(shift, torch.float32, "shift")
+    if weight.numel() != H or H != resid.shape[1] or (shift is not None and shift.numel() != H):
+        raise KernelError("add_tanh_norm: weight and shift must have the stream's width")
+    if rows is not None:
+        _want(rows, torch.int32, "rows")
+    _run("add_tanh_norm", lib().bf_add_tanh_norm, _ptr(resid), _ptr(delta), _ptr(delta2),
+         _ptr(bias), _c_float(alpha), _ptr(weight), _ptr(shift), _ptr(out), _ptr(rows), _c_int(n),
+         _c_int(H), _c_int(_dtype_code(out)), _c_int(1 if write_back else 0), _stream())
+
+
+def stream_pair(resid: torch.Tensor, delta: Optional[torch.Tensor],
+                delta2: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+                table: torch.Tensor, ids: torch.Tensor, scale: float, pair: torch.Tensor,
+                err: torch.Tensor) -> None:
+    """pair[t] = [resid[t] + delta[t] + delta2[t] + bias | table[ids[t]] * scale] in ``pair``'s
+    type (which is the table's); the stream is left as it is."""
+    _stream_deltas("stream_pair", resid, (delta, delta2), bias, pair.dtype)
+    _want(ids, torch.int32, "ids")
+    T, H = resid.shape
+    if (tuple(pair.shape) != (T, 2 * H) or not pair.is_contiguous() or table.dtype != pair.dtype
+            or table.shape[1] != H or not table.is_contiguous()):
+        raise KernelError("stream_pair: pair must be contiguous [T, 2 H] of the table's type")
+    _run("stream_pair", lib().bf_stream_pair, _ptr(resid), _ptr(delta), _ptr(delta2), _ptr(bias),
+         _ptr(table), _ptr(ids), _c_int(table.shape[0]), _c_float(scale), _ptr(pair), _c_int(T),
+         _c_int(H), _c_int(_dtype_code(pair)), _ptr(err), _stream())
 
 
 class RowScale:
@@ -196,18 +260,24 @@ FUSED_ACTIVATIONS = ("silu", "clamped")     # those that a product applies in it
 
 
 def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str,
-                  limit: float = 0.0, slope: float = 1.0, up_offset: float = 0.0) -> None:
+                  limit: float = 0.0, slope: float = 1.0, up_offset: float = 0.0,
+                  bias: Optional[torch.Tensor] = None) -> None:
     """out[t, c] = act(gate_up[t, c]) * gate_up[t, I + c]; ``activation`` one of
     ``GATE_ACTIVATIONS``.  "clamped": with g = min(gate, limit) and u = clamp(up, -limit, limit)
-    the result is g sigmoid(slope g) (u + up_offset)."""
+    the result is g sigmoid(slope g) (u + up_offset).  ``bias`` (float32 ``[2 I]``) is added to
+    the rows of ``gate_up`` first."""
     T, I = out.shape
+    if bias is not None:
+        _want(bias, torch.float32, "bias")
+        if bias.numel() != 2 * I:
+            raise KernelError("gated_act_mul: bias must have 2 I numbers")
     if activation not in GATE_ACTIVATIONS:
         raise KernelError(f"gated_act_mul: unknown activation {activation!r}")
     if gate_up.shape != (T, 2 * I) or not gate_up.is_contiguous() or gate_up.dtype != out.dtype:
         raise KernelError("gated_act_mul: gate_up must be contiguous [T, 2*I] of the output's dtype")
     _run("gated_act_mul", lib().bf_gated_act_mul, _ptr(gate_up), _ptr(out), _c_int(T), _c_int(I),
          _c_int(GATE_ACTIVATIONS[activation]), _c_int(_dtype_code(out)), _c_float(limit),
-         _c_float(slope), _c_float(up_offset), _stream())
+         _c_float(slope), _c_float(up_offset), _ptr(bias), _stream())
 
 
 def copy_ids(dst: torch.Tensor, src: torch.Tensor, pairs: torch.Tensor, n: int) -> None:
@@ -531,7 +601,8 @@ def conv_encode(proj: torch.Tensor, conv_w: Optional[torch.Tensor], taps: int,
                 err: torch.Tensor, pre_factor: Optional[torch.Tensor] = None,
                 pre_weight: Optional[torch.Tensor] = None, rot_magnitude: float = 1.0,
                 head_weight: Optional[torch.Tensor] = None,
-                q_head_scale: Optional[torch.Tensor] = None) -> None:
+                q_head_scale: Optional[torch.Tensor] = None,
+                proj_bias: Optional[torch.Tensor] = None) -> None:
     """``proj`` rows hold ``[q: nh dk | k: nkv dk | v: nkv dv]`` (a column block of a wider
     buffer is fine).  Per channel a causal convolution over the request's tokens with
     ``conv_w`` float32 ``[channels, taps]`` (``taps`` 0: none), whose reach behind the
@@ -544,8 +615,14 @@ def conv_encode(proj: torch.Tensor, conv_w: Optional[torch.Tensor], taps: int,
     over a whole projection: :func:`section_rms` takes the factors).  ``rot_magnitude``
     multiplies cosines and sines.  ``head_weight`` float32 ``[2, dk]``: behind the heads' norm,
     every q head is multiplied by the first row and every k head by the second.
-    ``q_head_scale`` float32 ``[nh]``: q head h is multiplied by its number."""
+    ``q_head_scale`` float32 ``[nh]``: q head h is multiplied by its number.  ``proj_bias``
+    float32 ``[channels]``: added to the projections first (``taps`` 0 only)."""
     T = proj.shape[0]
+    if proj_bias is not None:
+        _want(proj_bias, torch.float32, "proj_bias")
+        if proj_bias.numel() != nh * dk + nkv * (dk + dv) or taps:
+            raise KernelError("conv_encode: proj_bias must have one number per channel, and goes "
+                              "without a convolution")
     if head_weight is not None:
         _want(head_weight, torch.float32, "head_weight")
         if tuple(head_weight.shape) != (2, dk) or not head_weight.is_contiguous():
@@ -590,7 +667,7 @@ def conv_encode(proj: torch.Tensor, conv_w: Optional[torch.Tensor], taps: int,
          _c_int(nh), _c_int(nkv), _c_int(dk), _c_int(dv), _c_int(page_size), _c_ll(num_slots),
          _c_int(1 if unit_norm else 0), _c_float(eps), _c_int(_dtype_code(proj)), _ptr(table),
          _ptr(err), _ptr(pre_factor), _ptr(pre_weight), _c_float(rot_magnitude),
-         _ptr(head_weight), _ptr(q_head_scale), _stream())
+         _ptr(head_weight), _ptr(q_head_scale), _ptr(proj_bias), _stream())
 
 
 def conv_state_shift(proj: torch.Tensor, state: torch.Tensor, state_slots: torch.Tensor,
@@ -1005,12 +1082,34 @@ def moe_route(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, shared_g
          _c_int(1 if normalize else 0), _stream())
 
 
+class ExpertAct:
+    """The experts' activation: "silu", or "clamped" with its constants as in ``gated_act_mul``;
+    the shared expert's limit may be another one."""
+    __slots__ = ("activation", "limit", "shared_limit", "slope", "up_offset")
+
+    def __init__(self, activation: str = "silu", limit: float = 0.0, shared_limit: float = 0.0,
+                 slope: float = 1.0, up_offset: float = 0.0):
+        if activation not in FUSED_ACTIVATIONS:
+            raise KernelError(f"experts: activation {activation!r} is not supported")
+        self.activation, self.limit, self.shared_limit = activation, limit, shared_limit
+        self.slope, self.up_offset = slope, up_offset
+
+    def args(self):
+        return (_c_int(GATE_ACTIVATIONS[self.activation]), _c_float(self.limit),
+                _c_float(self.shared_limit), _c_float(self.slope), _c_float(self.up_offset))
+
+
+SILU_EXPERTS = ExpertAct()
+
+
 def moe_act(gu: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor, experts: int,
-            ff: int, shared_gate: Optional[bool] = None) -> None:
+            ff: int, shared_gate: Optional[bool] = None,
+            expert_act: ExpertAct = SILU_EXPERTS) -> None:
     """``act[t, c] = silu(gu[t, c]) * gu[t, F + c] * route_w[t, expert(c)]`` with
     ``expert(c) = c // ff`` for ``c < experts * ff``; the columns behind the experts' (a shared
     expert) take column ``experts`` of ``route_w`` when ``shared_gate``, else the weight one
-    (None: when ``route_w`` has exactly one column more than there are experts)."""
+    (None: when ``route_w`` has exactly one column more than there are experts).
+    ``expert_act``: another activation in silu's place."""
     T, F = act.shape
     _want(route_w, torch.float32, "route_w")
     if tuple(gu.shape) != (T, 2 * F) or not gu.is_contiguous() or not act.is_contiguous() \
@@ -1020,7 +1119,7 @@ def moe_act(gu: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor, experts:
         shared_gate = route_w.shape[1] == experts + 1
     _run("moe_act", lib().bf_moe_act, _ptr(gu), _ptr(route_w), _ptr(act), _c_int(T), _c_int(F),
          _c_int(experts), _c_int(ff), _c_int(route_w.shape[1]), _c_int(1 if shared_gate else 0),
-         _c_int(_dtype_code(act)), _stream())
+         _c_int(_dtype_code(act)), *expert_act.args(), _stream())
 
 
 def moe_identity_add(out: torch.Tensor, h: torch.Tensor, route_w: torch.Tensor, col: int) -> None:
@@ -1045,7 +1144,8 @@ def moe_sparse_takes(width: int, ff: int, ff_sh: int, top: int) -> bool:
 def moe_sparse(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                top_ids: torch.Tensor, top_w: torch.Tensor, route_w: torch.Tensor,
                out: torch.Tensor, experts: int, ff: int, ff_sh: int, top: int,
-               shared_gate: Optional[bool] = None, identity_col: int = -1) -> None:
+               shared_gate: Optional[bool] = None, identity_col: int = -1,
+               expert_act: ExpertAct = SILU_EXPERTS) -> None:
     """The mixture's output for a step of very few tokens, reading only the experts that
     were chosen (and the shared one): ``w_gate_up [2 F, width]`` and ``w_down [width, F]`` are
     the stacked weights (``F = experts * ff + ff_sh``), ``top_ids``/``top_w``/``route_w`` what
@@ -1071,7 +1171,7 @@ def moe_sparse(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
          _ptr(w_down), _ptr(top_ids), _ptr(top_w), _ptr(route_w), _c_int(route_w.shape[1]),
          _ptr(act), _ptr(out), _c_int(T), _c_int(width), _c_int(experts), _c_int(ff),
          _c_int(ff_sh), _c_int(top), _c_int(_dtype_code(h)), _c_int(1 if shared_gate else 0),
-         _c_int(identity_col), _stream())
+         _c_int(identity_col), *expert_act.args(), _stream())
     global _launches
     _launches += 1          # two kernels
 
@@ -1326,7 +1426,7 @@ LATENT_ROWS, LATENT_KEYS = 32, 64
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tensor,
                      positions: torch.Tensor, tables: torch.Tensor, out: torch.Tensor, B: int,
                      max_tokens: int, H: int, rank: int, scale: float, err: torch.Tensor,
-                     max_ctx: int = 0) -> None:
+                     max_ctx: int = 0, sinks: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention of query rows ``q [T, H, W]`` (already in the latent's
     coordinates) over a cache of one row ``[latent (rank) | shared key part]`` of ``W`` numbers
     per token, whose first ``rank`` numbers are also the value: ``out [T, H, rank]``, on the
@@ -1334,8 +1434,13 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tensor
     rows ``q_start[b] .. q_start[b+1]-1``, at most ``max_tokens`` of them.  ``max_ctx``: the
     longest context in the batch, if the caller knows it: a step with few rows then shares
     each request's key tiles out over several CTAs whose partial results a second kernel
-    makes one."""
+    makes one.  ``sinks`` (float32 ``[H]``): a learned logit per head in the softmax's
+    denominator."""
     W = q.shape[-1]
+    if sinks is not None:
+        _want(sinks, torch.float32, "sinks")
+        if sinks.numel() != H:
+            raise KernelError("latent_attention: sinks must have one number per head")
     if not latent_attention_takes(q.dtype, rank, W - rank):
         raise KernelError("latent_attention: bfloat16, a latent of a multiple of 16 up to 512, "
                           "with the shared part at most 640")
@@ -1359,7 +1464,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tensor
          _ptr(positions), _ptr(tables), _c_int(tables.stride(0)), _ptr(out), _c_int(B),
          _c_int(max_rows), _c_int(H), _c_int(W), _c_int(rank), _c_int(cache.shape[2]),
          _c_int(cache.shape[0]), _c_float(scale), _ptr(part_o), _ptr(part_ml), _c_int(splits),
-         _ptr(err), _stream())
+         _ptr(sinks), _ptr(err), _stream())
 
 
 # ------------------------------------------------------------- matrix products
@@ -1611,11 +1716,12 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Te
 def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Tensor,
                    bn: int = 0, gated: bool = False, accumulate: bool = False,
                    activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
-                   up_offset: float = 0.0) -> bool:
+                   up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None) -> bool:
     """out[M, N] = x[M, K] @ w[N, K]^T on pairs of SMs (``tcgen05.mma.cta_group::2``, tiles of
     256 token rows): the product for many token rows.  ``gated``: ``w`` is the stacked
     ``[2 N, K]`` gate/up weight and ``out[M, N] = silu(x w_gate^T) * (x w_up^T)``, bfloat16
     only; ``activation`` "clamped" with its constants as in ``gated_act_mul`` in silu's place.
+    ``gate_bias`` (float32 ``[2 N]``) is added to the sums before the activation.
     ``accumulate``: ``out`` (float32) ``+=`` the product.  ``bn``: accumulator columns
     per tile (0: chosen by the library).  Returns False, having done nothing, for shapes the
     kernel does not take."""
@@ -1638,8 +1744,16 @@ def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: tor
          _c_int(_dtype_code(out)),
          _c_int((2 if activation == "clamped" else 1) if gated else 0),
          _c_int(1 if accumulate else 0), _c_int(bn), _c_int(num_sms(x.device)), _ptr(err),
-         _c_float(limit), _c_float(slope), _c_float(up_offset), _stream())
+         _c_float(limit), _c_float(slope), _c_float(up_offset), _gate_bias(gate_bias, w), _stream())
     return True
+
+
+def _gate_bias(bias: Optional[torch.Tensor], w: torch.Tensor):
+    if bias is not None:
+        _want(bias, torch.float32, "gate_bias")
+        if bias.numel() != w.shape[0]:
+            raise KernelError("gated product: gate_bias must have one number per weight row")
+    return _ptr(bias)
 
 
 def gemm_cluster_plan(features: int, K: int, device: torch.device):
@@ -1764,7 +1878,7 @@ def gemm_swiglu_plan(inter: int, K: int, device: torch.device):
 def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor,
                      err: torch.Tensor, bn: int, row_scale: Optional[RowScale] = None,
                      activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
-                     up_offset: float = 0.0) -> bool:
+                     up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None) -> bool:
     """``silu_mul(x @ w_gate_up^T)`` as one kernel for at most 64 token rows: ``w_gate_up`` is
     ``[2 I, K]`` with the gate rows first, ``out`` is ``[M, I]``.  ``activation`` "clamped" with its
     constants as in ``gated_act_mul`` in silu's place.  Returns False, having done
@@ -1783,7 +1897,7 @@ def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor
          _c_int(I), _c_int(K), _c_ll(x.stride(0)), _c_ll(w_gate_up.stride(0)), _c_int(bn),
          _ptr(out), _c_ll(out.stride(0)), *_row_scale_args(row_scale, M), _ptr(err),
          _c_int(GATE_ACTIVATIONS[activation]), _c_float(limit), _c_float(slope),
-         _c_float(up_offset), _stream())
+         _c_float(up_offset), _gate_bias(gate_bias, w_gate_up), _stream())
     return True
 
 

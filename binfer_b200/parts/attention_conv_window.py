@@ -9,7 +9,8 @@ optionally each q and k head divided by its root mean square, after the rotation
 into the pages; scores with an optional soft cap; attention in
 which position i sees j <= i with ``i - j < window`` or ``j < keep_first`` (kept tokens stay
 at their true positions) and whose softmax has a learned logit per head in its denominator;
-the output projection.  Every key, also those of the step's own tokens, is read from the
+the output projection.  The q, k and v projections may have biases (without a convolution), which
+are added in float behind the product.  Every key, also those of the step's own tokens, is read from the
 pages, so portions can share a step with decoded tokens.
 
 Three more things a spec may ask for: a weight behind the heads' norm (``dim`` numbers for q
@@ -82,7 +83,10 @@ class ConvWindowAttention(Mixer):
         self.names = dict(spec.names)
         self.in_rows, self.out_cols = self.channels, self.H * self.dv
         self.w_in = self.w_out = self.conv_w = self.sinks = self.proj_norm_w = None
-        self.head_w = self.temp = self.bias_slope = self.bias_rate = None
+        self.head_w = self.temp = self.bias_slope = self.bias_rate = self.proj_bias = None
+        if spec.proj_bias and (self.taps or spec.proj_norm):
+            raise ValueError("biases of the projections go without a convolution and without a "
+                             "norm over a whole projection")
 
     # ----------------------------------------------------------------- weights
     def _spec(self, role: str) -> ParamSpec:
@@ -104,6 +108,10 @@ class ConvWindowAttention(Mixer):
             return ParamSpec(self.prefix + self.names[role],
                              (self.q_size if role == "q_norm" else self.k_size,), init="norm",
                              role="vector")
+        if role in ("q.bias", "k.bias", "v.bias"):
+            src = role[0]
+            return ParamSpec(self.prefix + self.names[src] + self.spec.bias_suffix, base[src][:1],
+                             init="around_zero", role="vector")
         src = role[:-5]                          # "q.conv" -> q
         return ParamSpec(self.prefix + self.names[src] + self.spec.conv_suffix,
                          (base[src][0], self.taps), init="conv", role="vector")
@@ -112,6 +120,8 @@ class ConvWindowAttention(Mixer):
         roles = ["q", "k", "v", "o"]
         if self.taps:
             roles += ["q.conv", "k.conv", "v.conv"]
+        if self.spec.proj_bias:
+            roles += ["q.bias", "k.bias", "v.bias"]
         if self.spec.sinks:
             roles.append("sink")
         if self.spec.proj_norm:
@@ -133,6 +143,8 @@ class ConvWindowAttention(Mixer):
         self.w_out = g("o")
         if self.taps:
             self.conv_w = torch.cat([g("q.conv"), g("k.conv"), g("v.conv")], dim=0).contiguous()
+        if self.spec.proj_bias:
+            self.proj_bias = torch.cat([g("q.bias"), g("k.bias"), g("v.bias")]).contiguous()
         if self.spec.sinks:
             self.sinks = g("sink")
         if self.spec.proj_norm:
@@ -172,7 +184,7 @@ class ConvWindowAttention(Mixer):
         inv = self.position.inv_freq if self.position is not None else None
         state = view.state if self.taps > 1 else None
         factors = None
-        if s.proj_norm:
+        if s.proj_norm:                 # (of the projections as they are: with no bias)
             factors = torch.empty((T, 2), dtype=torch.float32, device=proj.device)
             ops.section_rms(proj, 0, self.q_size, self.q_size, self.k_size, s.norm_eps, factors)
         ops.conv_encode(proj, self.conv_w, self.taps, state, ctx.state_slots, ctx.seq_of_token,
@@ -180,7 +192,8 @@ class ConvWindowAttention(Mixer):
                         view.v_cache, self.H, self.G, self.dk, self.dv, s.unit_norm, s.norm_eps,
                         ctx.err, pre_factor=factors, pre_weight=self.proj_norm_w,
                         rot_magnitude=getattr(self.position, "magnitude", 1.0),
-                        head_weight=self.head_w, q_head_scale=self.temp)
+                        head_weight=self.head_w, q_head_scale=self.temp,
+                        proj_bias=self.proj_bias)
         if self.taps > 1:
             ops.conv_state_shift(proj, state, ctx.state_slots, ctx.q_start, ctx.B, self.taps)
         keep = s.keep_first if s.window is not None else 0

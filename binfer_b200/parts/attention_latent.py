@@ -4,7 +4,8 @@ A down projection of the mixer's input yields ``rank + dr`` numbers per token: t
 ``rank``, RMS-normed with a weight, are the latent ``c``; the last ``dr``, rotated by the
 token's position, are a key part that all heads share.  Head h's key is ``[W_uk,h c | shared
 part]``, its value ``W_uv,h c``, its query ``[d plain | dr rotated]``; scores are scaled,
-masked causally and pass an ordinary softmax; each head's output may be multiplied by the
+masked causally and pass an ordinary softmax (whose denominator may hold a learned logit per
+head, ``sinks``); each head's output may be multiplied by the
 sigmoid of one projected number per head; the output projection follows.
 
 Only ``c`` and the shared key part are cached: one cache "head" of ``rank + dr`` numbers per
@@ -66,23 +67,27 @@ class LatentAttention(Mixer):
         self.names = dict(s.names)
         self.gate_off = self.q_rows + self.kv_size
         self.w_proj = self.w_ukT = self.w_uv = self.w_o = self.norm_w = None
-        self.w_uq = self.q_norm_w = None
+        self.w_uq = self.q_norm_w = self.sinks = None
 
     # ----------------------------------------------------------------- weights
     def _spec(self, role: str) -> ParamSpec:
-        n = self.prefix + self.names[role]
         shape = {"q": (self.q_size, self.hidden), "dkv": (self.kv_size, self.hidden),
                  "dkv_norm": (self.rank,), "uk": (self.H * self.d, self.rank),
                  "uv": (self.H * self.dv, self.rank), "g": (self.H, self.hidden),
                  "o": (self.hidden, self.H * self.dv), "dq": (self.q_rank, self.hidden),
-                 "dq_norm": (self.q_rank,), "uq": (self.q_size, self.q_rank)}[role]
+                 "dq_norm": (self.q_rank,), "uq": (self.q_size, self.q_rank),
+                 "sink": (self.H,)}[role]
+        n = self.prefix + self.names[role]
+        if role == "sink":
+            return ParamSpec(n, shape, init="around_zero", role="vector")
         if role in ("dkv_norm", "dq_norm"):
             return ParamSpec(n, shape, init="norm", role="vector")
         return ParamSpec(n, shape)
 
     def _roles(self) -> List[str]:
         q = ["dq", "dq_norm", "uq"] if self.q_rank else ["q"]
-        return q + ["dkv", "dkv_norm", "uk", "uv"] + (["g"] if self.spec.head_gate else []) + ["o"]
+        return (q + ["dkv", "dkv_norm", "uk", "uv"] + (["g"] if self.spec.head_gate else [])
+                + (["sink"] if self.spec.sinks else []) + ["o"])
 
     def param_specs(self) -> List[ParamSpec]:
         return [self._spec(r) for r in self._roles()]
@@ -100,6 +105,8 @@ class LatentAttention(Mixer):
         self.w_ukT = g("uk").view(self.H, self.d, self.rank).transpose(1, 2).contiguous()
         self.w_uv = g("uv").view(self.H, self.dv, self.rank).contiguous()
         self.w_o = g("o")
+        if self.spec.sinks:
+            self.sinks = g("sink")
 
     # ------------------------------------------------------------------- cache
     def kv_need(self) -> Optional[KVNeed]:
@@ -135,13 +142,14 @@ class LatentAttention(Mixer):
             ops.latent_attention(q_abs, view.k_cache, ctx.q_start, ctx.positions,
                                  ctx.block_tables[g], o_lat, ctx.B,
                                  1 if ctx.decode_only else ctx.max_q_len, H, self.rank,
-                                 s.softmax_scale, ctx.err, max_ctx=ctx.max_ctx_len)
+                                 s.softmax_scale, ctx.err, max_ctx=ctx.max_ctx_len,
+                                 sinks=self.sinks)
         else:
             ops.paged_attention_generic(
                 q_abs.view(T, H * self.kv_size), view.k_cache, view.k_cache, ctx.seq_of_token,
                 ctx.positions, ctx.block_tables[g], o_lat.view(T, H * self.rank), H, 1,
                 self.kv_size, None, s.softmax_scale, ctx.err, value_dim=self.rank,
-                v_stride=self.kv_size)
+                v_stride=self.kv_size, sinks=self.sinks)
         out = torch.empty((T, H, self.dv), dtype=x.dtype, device=x.device)
         linear_heads(o_lat, self.w_uv, out)
         out = out.view(T, H * self.dv)

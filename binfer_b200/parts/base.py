@@ -165,17 +165,21 @@ class EntryView:
 
 
 class DeferredLinear:
-    """``x @ w^T`` not yet computed: how a part may hand its output to the block
+    """``x @ w^T (+ bias)`` not yet computed: how a part may hand its output to the block
     (``forward_deferred``), so that the product can be fused with what follows it, the add
-    into the residual stream and the next norm."""
-    __slots__ = ("x", "w")
+    into the residual stream and the next norm.  ``bias``: float32, one number per output."""
+    __slots__ = ("x", "w", "bias")
 
-    def __init__(self, x: torch.Tensor, w: torch.Tensor):
-        self.x, self.w = x, w
+    def __init__(self, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None):
+        self.x, self.w, self.bias = x, w, bias
 
     def compute(self) -> torch.Tensor:
         from .linear import linear
-        return linear(self.x, self.w)
+        y = linear(self.x, self.w)
+        if self.bias is not None:
+            from ..csrc import ops
+            ops.bias_add(y, self.bias)
+        return y
 
 
 class ScaledRows:
@@ -213,28 +217,39 @@ class ResidualStream:
         self.x = x
         self.pending: Optional[torch.Tensor] = None
         self.pending2: Optional[torch.Tensor] = None     # see add_pair
+        # float32 vector that goes with ``pending``: the bias of the product that made it
+        self.pending_bias: Optional[torch.Tensor] = None
         self.ready = None                # a tensor, or ScaledRows
         self.ready_for = None
         # the stream itself in the activation type, for sublayers that read it without a
         # norm in front; kept by the kernel that last changed the stream, dropped by any other
         self.reading: Optional[torch.Tensor] = None
 
-    def add(self, delta: torch.Tensor) -> None:
+    def add(self, delta: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
         if self.pending is not None or self.pending2 is not None:
             self.flush()
-        self.pending = delta
+        self.pending, self.pending_bias = delta, bias
         self.ready = self.ready_for = None
         self.reading = None
 
-    def add_pair(self, a: torch.Tensor, b: torch.Tensor) -> None:
+    def add_pair(self, a: torch.Tensor, b: torch.Tensor,
+                 bias: Optional[torch.Tensor] = None) -> None:
         """Two sublayer outputs at once (sublayers that ran side by side on one norm's
-        output).  A norm that takes a second delta (``forward(..., also=)``) folds both in
-        one pass; before any other reader :meth:`flush` adds them."""
-        self.add(a)
+        output), and a bias of theirs.  A norm that takes a second delta (``forward(...,
+        also=)``) folds both in one pass; before any other reader :meth:`flush` adds them."""
+        self.add(a, bias)
         self.pending2 = b
+
+    def replace(self, x: torch.Tensor) -> None:
+        """A new stream in the old one's place (its pending adds went into what made ``x``)."""
+        self.x = x
+        self.pending = self.pending2 = self.pending_bias = None
+        self.ready = self.ready_for = self.reading = None
 
     def norm_input(self, norm, rows: Optional[torch.Tensor] = None, n_rows: int = 0):
         """``norm`` over the stream with everything pending folded in."""
+        if self.pending_bias is not None and not getattr(norm, "takes_pending_bias", False):
+            self.flush()
         if self.pending2 is not None:
             if getattr(norm, "takes_second_delta", False):
                 also, self.pending2 = self.pending2, None
@@ -266,7 +281,8 @@ class ResidualStream:
         from .linear import linear_add_norm
         fs = getattr(norm, "fused_scale", None)
         self.reading = None
-        if fs is not None and getattr(consumer, "accepts_scaled_rows", False):
+        if (fs is not None and getattr(consumer, "accepts_scaled_rows", False)
+                and d.bias is None):
             self.flush()
             weight, eps = fs()
             got = linear_add_norm(d.x, d.w, self.x, weight, eps)
@@ -278,8 +294,8 @@ class ResidualStream:
     def flush(self) -> None:
         from ..csrc import ops
         if self.pending is not None:
-            ops.residual_add(self.x, self.pending)
-            self.pending = None
+            ops.residual_add(self.x, self.pending, self.pending_bias)
+            self.pending = self.pending_bias = None
         if self.pending2 is not None:
             ops.residual_add(self.x, self.pending2)
             self.pending2 = None

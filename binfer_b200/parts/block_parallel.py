@@ -12,6 +12,7 @@ from typing import List
 from ..config.specs import LayerSpec, NameLayout
 from .base import (BuildEnv, EntryView, Part, ResidualStream, StepContext, build_ffn,
                    build_mixer, build_norm, register_block)
+from .linear import linear
 
 
 class ParallelBlock(Part):
@@ -38,10 +39,15 @@ class ParallelBlock(Part):
     def forward(self, stream: ResidualStream, ctx: StepContext, view: EntryView) -> None:
         h = stream.norm_input(self.norm)
         y = self.mixer.forward(h, ctx, view)
-        if self.ffn is not None:
+        if self.ffn is None:
+            stream.add(y)
+            return
+        deferred = getattr(self.ffn, "forward_deferred", None)
+        if deferred is None:
             stream.add_pair(y, self.ffn.forward(h, ctx))
         else:
-            stream.add(y)
+            d = deferred(h, ctx)        # (its bias rides on the adds)
+            stream.add_pair(y, linear(d.x, d.w), d.bias)
 
 
 register_block("parallel", ParallelBlock)

@@ -1,7 +1,9 @@
 """Dense gated feed-forward: ``down( act(gate(x)) * up(x) )``, ``act`` silu (SwiGLU) or the
 tanh form of gelu, or the clamped form ``min(g, c) sigmoid(a min(g, c)) (clamp(u, -c, c) + b)``
 with three constants (``GatedMLPSpec.activation``; silu and the clamped form run in the products'
-epilogues where those kernels apply, else the product and the activation kernel run).
+epilogues where those kernels apply, else the product and the activation kernel run).  With
+``GatedMLPSpec.bias`` the three projections have biases: the first two are added (in float) where
+the activation is applied, the last one rides on the add into the residual stream.
 
 ``silu(g) = g / (1 + exp(-g))`` (cuda/kernels/bf16_kernels.cu:461-477).  The
 reference runs gate and up as two products (src/engine/batched_engine.ts:1243-1244);
@@ -39,24 +41,31 @@ class GatedMLP(FeedForward):
                          up_offset=spec.up_offset)
         if spec.activation == "clamped" and not spec.limit > 0:
             raise ValueError("a clamped activation needs a positive limit")
-        if spec.bias:
-            raise ValueError("feed-forward biases are not supported")
         self.spec, self.hidden, self.prefix, self.env = spec, hidden_size, prefix, env
         self.inter = spec.intermediate_size
         self.w_gate_up = self.w_down = None
+        self.b_gate_up = self.b_down = None     # float32, with GatedMLPSpec.bias
         self._swiglu_plan = None
 
     def param_specs(self) -> List[ParamSpec]:
         p = self.prefix
         gate, up, down = self.spec.names
-        return [ParamSpec(p + gate, (self.inter, self.hidden)),
-                ParamSpec(p + up, (self.inter, self.hidden)),
-                ParamSpec(p + down, (self.hidden, self.inter))]
+        specs = [ParamSpec(p + gate, (self.inter, self.hidden)),
+                 ParamSpec(p + up, (self.inter, self.hidden)),
+                 ParamSpec(p + down, (self.hidden, self.inter))]
+        if self.spec.bias:
+            specs += [ParamSpec(p + n, (size,), init="around_zero", role="vector")
+                      for n, size in zip(self.spec.bias_names,
+                                         (self.inter, self.inter, self.hidden))]
+        return specs
 
     def load(self, get: Callable[[ParamSpec], torch.Tensor]) -> None:
-        g, u, d = self.param_specs()
+        g, u, d, *biases = self.param_specs()
         self.w_gate_up = torch.cat([get(g), get(u)], dim=0).contiguous()
         self.w_down = get(d)
+        if biases:
+            bg, bu, bd = (get(b) for b in biases)
+            self.b_gate_up, self.b_down = torch.cat([bg, bu]).contiguous(), bd
 
     accepts_scaled_rows = True
 
@@ -65,17 +74,18 @@ class GatedMLP(FeedForward):
 
     def forward_deferred(self, x, ctx: StepContext) -> DeferredLinear:
         """Everything but the down projection (see ``GQAAttention.forward_deferred``)."""
-        if isinstance(x, ScaledRows) and (self.inter % 8 or self.inter < 256 or not self.silu):
+        if isinstance(x, ScaledRows) and (self.inter % 8 or self.inter < 256 or not self.silu
+                                          or self.spec.bias):
             x = x.dense()                  # the activation kernel takes the factor at other sizes only
         x, row_scale = split_scaled(x)
         h = torch.empty((x.shape[0], self.inter), dtype=x.dtype, device=x.device)
         if not self._project_fused(x, h, row_scale):
             gu = linear(x, self.w_gate_up)
-            if self.silu:
+            if self.silu and self.b_gate_up is None:
                 ops.silu_mul(gu, h, row_scale=row_scale)
             else:
-                ops.gated_act_mul(gu, h, **self._act)
-        return DeferredLinear(h, self.w_down)
+                ops.gated_act_mul(gu, h, bias=self.b_gate_up, **self._act)
+        return DeferredLinear(h, self.w_down, self.b_down)
 
     def _project_fused(self, x, h, row_scale) -> bool:
         """Few token rows in bfloat16: the stacked projection with the activation in its
@@ -87,7 +97,7 @@ class GatedMLP(FeedForward):
         if pair_from and x.shape[0] >= pair_from and row_scale is None:
             # many token rows: the product on pairs of SMs, the activation in its epilogue
             return ops.gemm_bf16_pair(x, self.w_gate_up, h, ops.error_word(x.device), gated=True,
-                                      **self._act)
+                                      gate_bias=self.b_gate_up, **self._act)
         if x.shape[0] > swiglu_token_limit():
             return False
         if self._swiglu_plan is None:
@@ -96,7 +106,7 @@ class GatedMLP(FeedForward):
         if not plan or plan[1] < FUSE_SWIGLU_FILL * ops.num_sms(x.device):
             return False
         return ops.gemm_bf16_swiglu(x, self.w_gate_up, h, ops.error_word(x.device), plan[0],
-                                    row_scale=row_scale, **self._act)
+                                    row_scale=row_scale, gate_bias=self.b_gate_up, **self._act)
 
 
 register_ffn("gated_mlp", GatedMLP)

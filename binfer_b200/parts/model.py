@@ -68,13 +68,22 @@ class DecoderModel:
                           ParamSpec(spec.pass_table[0], (int(spec.pass_table[1]), spec.hidden_size),
                                     init="around_zero", role="vector"))
         self.pass_table: Optional[torch.Tensor] = None
+        self.pass_proj_spec = (None if spec.pass_projection is None else
+                               ParamSpec(spec.pass_projection,
+                                         (spec.hidden_size, 2 * spec.hidden_size)))
+        self.pass_proj: Optional[torch.Tensor] = None
         for e, entry in enumerate(spec.schedule):
             if entry.before is not None and entry.before.row is not None and not (
                     self.pass_spec is not None
                     and 0 <= entry.before.row < self.pass_spec.shape[0]):
                 raise ValueError(f"schedule entry {e} adds row {entry.before.row} of a table "
                                  f"of pass vectors that the model lacks or that is shorter")
-            if (entry.before is not None and entry.before.embedding
+            if entry.before is not None and entry.before.project and (
+                    self.pass_proj_spec is None or entry.before.embedding
+                    or entry.before.row is not None):
+                raise ValueError(f"schedule entry {e} projects the stream: the model needs a pass "
+                                 f"projection, and nothing else is added there")
+            if (entry.before is not None and (entry.before.embedding or entry.before.project)
                     and spec.position_vectors is not None):
                 raise ValueError("the embedding output cannot be added again where positions "
                                  "add vectors to it")
@@ -95,6 +104,8 @@ class DecoderModel:
         specs += self.final_norm.param_specs()
         if self.pass_spec is not None:
             specs.append(self.pass_spec)
+        if self.pass_proj_spec is not None:
+            specs.append(self.pass_proj_spec)
         if self.head_spec is not None:
             specs.append(self.head_spec)
         return specs
@@ -115,6 +126,8 @@ class DecoderModel:
         self.final_norm.load(get)
         if self.pass_spec is not None:
             self.pass_table = get(self.pass_spec)
+        if self.pass_proj_spec is not None:
+            self.pass_proj = get(self.pass_proj_spec)
         self.lm_head = self.embed if self.head_spec is None else get(self.head_spec)
 
     def weight_bytes(self) -> int:
@@ -200,10 +213,18 @@ class DecoderModel:
     def _open_pass(self, stream: ResidualStream, ctx: StepContext, before) -> None:
         """Fold the pending sublayer output into the stream together with what a pass starts
         with: the embedding output again (gathered from the table anew, in float) and a row
-        of the pass table."""
+        of the pass table; or replace the stream by the pass projection of itself and the
+        embedding output."""
+        if before.project:
+            pair = torch.empty((ctx.T, 2 * self.spec.hidden_size), dtype=self.env.dtype,
+                               device=self.env.device)
+            ops.stream_pair(stream.x, stream.pending, stream.pending2, stream.pending_bias,
+                            self.embed, ctx.token_ids, self.spec.embedding_scale, pair, ctx.err)
+            stream.replace(linear(pair, self.pass_proj, out_dtype=torch.float32))
+            return
         if not before.embedding and before.row is None:
             return
-        if stream.pending2 is not None:
+        if stream.pending2 is not None or stream.pending_bias is not None:
             stream.flush()
         delta, stream.pending = stream.pending, None
         stream.ready = stream.ready_for = stream.reading = None

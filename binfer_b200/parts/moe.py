@@ -22,6 +22,9 @@ router adds their weights up in one column, and a small kernel adds input times 
 to the result.  A third way ("sigmoid") takes the sigmoids of the outputs as scores; a group may
 count by the sum of its few largest scores, and the chosen scores may stay as they are.
 
+``MoESpec.activation`` "clamped": ``min(g, c) sigmoid(a min(g, c)) (clamp(u, -c, c) + b)`` in silu's
+place, the shared expert with a limit c of its own.
+
 A step of very few tokens in bfloat16 (a request that decodes alone) would read every expert
 for nothing; there the chosen experts' rows alone are read, a warp per output row
 (``ops.moe_sparse``).  The float32 engine keeps the one path, so that its sums have one order.
@@ -46,8 +49,14 @@ SPARSE = os.environ.get("BINFER_B200_MOE_SPARSE", "1") != "0"
 
 class MoEFeedForward(FeedForward):
     def __init__(self, spec: MoESpec, hidden_size: int, prefix: str, env: BuildEnv):
-        if spec.activation != "silu":
-            raise ValueError(f"activation {spec.activation!r} is not supported (supported: 'silu')")
+        if spec.activation not in ops.FUSED_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not supported (supported: "
+                             f"{sorted(ops.FUSED_ACTIVATIONS)})")
+        if spec.activation == "clamped" and not (spec.limit > 0 and (
+                spec.shared_limit > 0 or not spec.shared_size)):
+            raise ValueError("clamped experts need positive limits")
+        self.expert_act = ops.ExpertAct(spec.activation, spec.limit, spec.shared_limit, spec.slope,
+                                        spec.up_offset)
         self.identity = int(getattr(spec, "identity", 0) or 0)
         if not 1 <= spec.top <= spec.num_experts + self.identity:
             raise ValueError("moe: top must be between 1 and the number of router outputs")
@@ -129,11 +138,12 @@ class MoEFeedForward(FeedForward):
             out = torch.empty((T, self.hidden), dtype=x.dtype, device=x.device)
             ops.moe_sparse(x, self.w_gate_up, self.w_down, top_ids, top_w, route_w, out, self.E,
                            self.ff, self.ff_sh, self.top, shared_gate=self.gated_shared,
-                           identity_col=self.id_col)
+                           identity_col=self.id_col, expert_act=self.expert_act)
             return out
         gu = linear(x, self.w_gate_up)
         act = torch.empty((T, self.F), dtype=x.dtype, device=x.device)
-        ops.moe_act(gu, route_w, act, self.E, self.ff, shared_gate=self.gated_shared)
+        ops.moe_act(gu, route_w, act, self.E, self.ff, shared_gate=self.gated_shared,
+                    expert_act=self.expert_act)
         out = linear(act, self.w_down)
         if self.identity:
             ops.moe_identity_add(out, x, route_w, self.id_col)

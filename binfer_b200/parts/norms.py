@@ -50,8 +50,8 @@ class RMSNorm(Norm):
         if rows is None and stream.ready_for is self:
             out, stream.ready, stream.ready_for = stream.ready, None, None
             return out           # the kernel before already prepared this norm
-        if stream.pending2 is not None:
-            stream.flush()       # a pair of adds: this norm's kernel folds one only
+        if stream.pending2 is not None or stream.pending_bias is not None:
+            stream.flush()       # a pair of adds or a bias: this norm's kernel folds one add only
         stream.ready = stream.ready_for = None
         n = n_rows if rows is not None else stream.x.shape[0]
         out = torch.empty((n, self.size), dtype=self.env.dtype, device=self.env.device)
@@ -125,6 +125,8 @@ class LayerNorm(Norm):
                 n_rows: int = 0, also: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Normed activations of every row, or of ``rows`` only (the stream is then left as it
         is).  ``also``: one more sublayer output to add beside the pending one."""
+        if stream.pending_bias is not None:
+            stream.flush()
         stream.ready = stream.ready_for = None
         n = n_rows if rows is not None else stream.x.shape[0]
         out = torch.empty((n, self.size), dtype=self.env.dtype, device=self.env.device)
@@ -137,3 +139,54 @@ class LayerNorm(Norm):
 
 
 register_norm("layernorm", LayerNorm)
+
+
+class TanhNorm(Norm):
+    """``y = tanh(alpha x) * w + b``: a norm that takes no statistic of the row (dynamic tanh);
+    alpha is a tensor of one number.  Folds the stream's pending add, a second one (``also``)
+    and the bias of the product that made them (``bias``) into the same pass."""
+
+    takes_second_delta = True      # forward(..., also=): see ResidualStream.add_pair
+    takes_pending_bias = True      # ... and the stream's pending bias
+
+    def __init__(self, spec: NormSpec, size: int, name: str, env: BuildEnv):
+        self.size, self.name, self.env = size, name, env
+        self.alpha_name = name + spec.alpha_suffix
+        self.bias_name = None if spec.bias_suffix is None else name + spec.bias_suffix
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self.alpha = 1.0
+
+    def param_specs(self) -> List[ParamSpec]:
+        specs = [ParamSpec(self.name, (self.size,), init="norm", role="vector"),
+                 ParamSpec(self.alpha_name, (), init="norm", role="vector")]
+        if self.bias_name is not None:
+            specs.append(ParamSpec(self.bias_name, (self.size,), init="around_zero",
+                                   role="vector"))
+        return specs
+
+    def load(self, get: Callable[[ParamSpec], torch.Tensor]) -> None:
+        specs = self.param_specs()
+        self.weight = get(specs[0])
+        self.alpha = float(get(specs[1]))          # one number: an argument of the kernels
+        self.bias = get(specs[2]) if len(specs) > 2 else None
+
+    def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None,
+                n_rows: int = 0, also: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Normed activations of every row, or of ``rows`` only (the stream is then left as it
+        is).  ``also``: one more sublayer output to add beside the pending one."""
+        if rows is None and also is None and stream.ready_for is self:
+            out, stream.ready, stream.ready_for = stream.ready, None, None
+            return out           # the kernel before already prepared this norm
+        stream.ready = stream.ready_for = None
+        n = n_rows if rows is not None else stream.x.shape[0]
+        out = torch.empty((n, self.size), dtype=self.env.dtype, device=self.env.device)
+        ops.add_tanh_norm(stream.x, stream.pending, also, stream.pending_bias, self.alpha,
+                          self.weight, self.bias, out, rows=rows, write_back=rows is None)
+        if rows is None:
+            stream.pending = stream.pending_bias = None
+            stream.reading = None
+        return out
+
+
+register_norm("tanh_norm", TanhNorm)
