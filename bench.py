@@ -372,6 +372,34 @@ def differential_config(size, layers=8):
                        for i in range(layers)]}
 
 
+def projected_config(size, layers=8):
+    """The design whose looped passes project the stream, at the Qwen3 shape of that name,
+    ``layers`` layer runs (an even number): latent attention with a dense feed-forward, windowed
+    attention and latent attention with a mixture, walked ``(layers - 2) / 3`` times, then one more
+    of latent and of windowed attention for what is left.  Windowed attention has the shape's
+    heads and a window of 1,024, latent attention as many heads, of 128 plain and 64 rotated
+    sizes, over a latent of 512; the dense feed-forward is the shape's, the mixture eight experts
+    of which two run, which with the shared expert are as many active inner features."""
+    width, heads, kv, d, ff = HYBRID_SIZES[size][:5]
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0},
+           "shared": {"ff": ff // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2}}
+    window = {"type": "attention", "mlp": moe,
+              "mixer": {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5,
+                        "mask": {"size": 1024}, "rot": {"base": 1e6, "dims": d}}}
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512,
+              "scale": 192 ** -0.5,
+              "rot": {"base": 1e4, "dims": 64, "scaling": {"factor": 4.0, "original": 4096,
+                                                           "fast": 32.0, "slow": 1.0}}}
+    looped = [{"type": "latent_attention", "mlp": dense, "mixer": latent}, window,
+              {"type": "latent_attention", "mlp": moe, "mixer": latent}]
+    times = max(1, (layers - 1) // 3)
+    tail = [looped[2], window] * layers
+    return {"architecture": "Nazorax", "vocab": 32000, "width": width, "norm": {"eps": 1e-5},
+            "layers": looped + tail[:max(0, layers - 3 * times)],
+            "loop": {"start": 0, "stop": 3, "times": times}}
+
+
 def hybrid_compare(args, design="hybrid"):
     """Prefill and decode throughput of the hybrid design (matrix-memory layers alternating
     with pooled-window attention layers), or with ``design`` "side_by_side" of the design
@@ -384,7 +412,7 @@ def hybrid_compare(args, design="hybrid"):
     import torch
     from binfer_b200 import Engine, Qwen3Config
     from binfer_b200.config import (FikotarConfig, FolivikConfig, GukidraConfig, KetopelConfig,
-                                    PabelixConfig)
+                                    NazoraxConfig, PabelixConfig)
     from binfer_b200.engine.runner import StepItem
     from binfer_b200.profiling import Profiler
     layers = args.layers or 8
@@ -392,10 +420,14 @@ def hybrid_compare(args, design="hybrid"):
     steps, warmup = min(args.steps, 64), max(args.warmup, 3)
     what = {"hybrid": "hybrid design", "side_by_side": "side-by-side design",
             "looped": "looped design", "state_space": "state space design",
-            "differential": "differential attention design"}[design]
+            "differential": "differential attention design",
+            "projected": "design with projected passes"}[design]
     # the design with state space layers stands beside the looped design, the closest one
     # (latent attention, a recurrence per head, softmax attention), not beside Qwen3
-    beside = "the looped design" if design == "state_space" else "the Qwen3 decoder"
+    # (and the one with projected passes beside that: both have latent and windowed attention
+    # and a mixture with a shared expert)
+    beside = ("the looped design" if design == "state_space" else
+              "the state space design" if design == "projected" else "the Qwen3 decoder")
     record = {"metric": what + " beside " + beside + " at equal layer sizes "
                         "(prefill of 2048 tokens; decode at batch %d, context %d)" % (B, context),
               "dtype": "bf16", "data": "synthetic", "layers": layers, "sizes": {}}
@@ -410,9 +442,13 @@ def hybrid_compare(args, design="hybrid"):
                 if design == "state_space"
                 else PabelixConfig.from_dict(differential_config(size, layers))
                 if design == "differential"
+                else NazoraxConfig.from_dict(projected_config(size, layers))
+                if design == "projected"
                 else FikotarConfig.from_dict(side_by_side_config(size, layers)))
         other = (("looped", KetopelConfig.from_dict(looped_config(size, layers)))
-                 if design == "state_space" else ("qwen3", Qwen3Config.from_dict(qwen)))
+                 if design == "state_space" else
+                 ("state_space", FolivikConfig.from_dict(state_space_config(size, layers)))
+                 if design == "projected" else ("qwen3", Qwen3Config.from_dict(qwen)))
         for name, cfg in ((design, ours), other):
             engine = Engine(cfg, "bfloat16", random_seed=0, num_pages=(B + 1) * (context // ps) + 64,
                             page_size=ps, max_seq_len=context, max_batch_size=B + 1,
@@ -566,9 +602,14 @@ def main():
     ap.add_argument("--differential", action="store_true",
                     help="the same for the design with differential attention, dense clamped "
                          "feed-forwards and a mixture of experts with a sigmoid router")
+    ap.add_argument("--projected", action="store_true",
+                    help="the same for the design whose looped passes project the stream with the "
+                         "embedding output (tanh norms, latent attention with sinks, windowed "
+                         "attention with biases, clamped experts); it stands beside the design "
+                         "with state space layers instead of Qwen3")
     ap.add_argument("--hybrid-sizes", default="",
-                    help="with --hybrid, --side-by-side, --looped, --state-space or "
-                         "--differential: 1.7b, 8b or both (default)")
+                    help="with --hybrid, --side-by-side, --looped, --state-space, --differential "
+                         "or --projected: 1.7b, 8b or both (default)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -587,6 +628,8 @@ def main():
         return hybrid_compare(args, "state_space")
     if args.differential:
         return hybrid_compare(args, "differential")
+    if args.projected:
+        return hybrid_compare(args, "projected")
     if args.profile:
         return profile_steps(args)
     if args.workload == "serve":

@@ -11,13 +11,15 @@ from .fikotar import FikotarConfig
 from .ketopel import KetopelConfig
 from .folivik import FolivikConfig
 from .pabelix import PabelixConfig
+from .nazorax import NazoraxConfig
 from .registry import (family_for, load_config, parse_config, read_config_json,
                        register_architecture, registered_architectures)
 
 __all__ = [
     "AttentionSpec", "ConfigError", "GatedMLPSpec", "LayerSpec", "ModelSpec", "NameLayout",
     "NormSpec", "RopeSpec", "ScheduleEntry", "ScoreSpec", "Qwen3Config",
-    "GukidraConfig", "FikotarConfig", "KetopelConfig", "FolivikConfig", "PabelixConfig", "DifferentialAttentionSpec",
+    "GukidraConfig", "FikotarConfig", "KetopelConfig", "FolivikConfig", "PabelixConfig", "NazoraxConfig",
+    "DifferentialAttentionSpec",
     "PositionVectorSpec", "Mamba2Spec", "GatedDeltaRuleSpec",
     "LatentAttentionSpec", "PassStart", "RampScaling", "ConvWindowAttentionSpec", "RetentionSpec", "MixerBranch",
     "ParallelMixersSpec", "MoESpec", "WavelengthScaling", "MLSTMSpec", "PooledWindowAttentionSpec", "family_for", "load_config",

@@ -260,8 +260,8 @@ BF_EXPORT int bf_residual_add(float* resid, const void* delta, long long n, int 
 // here they are the two halves of one fused projection's output row).
 // ACT: the activations of gate_act.cuh.  `bias` (2 I numbers, or null) is added to the row first.
 template <typename A, int ACT>
-__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, int T, int I,
-                                BfGateConst gk, const float* __restrict__ bias) {
+__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, long long ldo,
+                                int T, int I, BfGateConst gk, const float* __restrict__ bias) {
   const size_t n = (size_t)T * I;
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
@@ -273,7 +273,7 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ out, i
       g += bias[c];
       u += bias[I + c];
     }
-    bf_st(out + i, bf_gate_mul<ACT>(g, u, gk));
+    bf_st(out + t * ldo + c, bf_gate_mul<ACT>(g, u, gk));
   }
 }
 
@@ -328,8 +328,8 @@ __global__ void silu_mul_bf16_scaled_kernel(const __nv_bfloat16* __restrict__ gu
 // bf16, I a multiple of 8: eight elements per thread with 16-byte loads and stores.
 template <int ACT>
 __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
-                                         __nv_bfloat16* __restrict__ out, int T, int I,
-                                         BfGateConst gk, const float* __restrict__ bias) {
+                                         __nv_bfloat16* __restrict__ out, long long ldo, int T,
+                                         int I, BfGateConst gk, const float* __restrict__ bias) {
   BF_TRACE_POINT(10 * BF_TR_SILU);
   bf_pdl_trigger();
   bf_pdl_wait();
@@ -368,7 +368,7 @@ __global__ void silu_mul_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
         o2[j] = __floats2bfloat162_rn(bf_gate_mul_fast<ACT>(g.x, u.x, gk),
                                       bf_gate_mul_fast<ACT>(g.y, u.y, gk));
       }
-      *reinterpret_cast<uint4*>(out + (k ? t2 * I + c2 : t * I + c)) = o4;
+      *reinterpret_cast<uint4*>(out + (k ? t2 * ldo + c2 : t * ldo + c)) = o4;
     }
   }
 }
@@ -391,46 +391,49 @@ BF_EXPORT int bf_silu_mul_scaled(const void* gu, void* out, int T, int I,
 }
 
 template <int ACT>
-static int gated_act_mul_launch(const void* gu, void* out, int T, int I, int act_dtype,
+static int gated_act_mul_launch(const void* gu, void* out, long long ldo, int T, int I, int act_dtype,
                                 cudaStream_t stream, BfGateConst gk = BfGateConst(),
                                 const float* bias = nullptr) {
   if (T <= 0) return 0;
   const int threads = 256;
-  if (act_dtype == BF_DTYPE_BF16 && I % 8 == 0 && ((uintptr_t)gu & 15) == 0 &&
+  if (act_dtype == BF_DTYPE_BF16 && I % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)gu & 15) == 0 &&
       ((uintptr_t)out & 15) == 0 && ((uintptr_t)bias & 7) == 0) {
     long long blocks = ((long long)T * (I / 8) + threads - 1) / threads;
     if (blocks > 148 * 16) blocks = 148 * 16;
     return bf_launch_pdl(silu_mul_bf16_vec_kernel<ACT>, dim3((int)blocks), dim3(threads), 0,
-                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk, bias);
+                         stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ldo, T, I, gk,
+                         bias);
   }
   long long blocks = ((long long)T * I + threads - 1) / threads;
   if (blocks > 148 * 32) blocks = 148 * 32;
   if (act_dtype == BF_DTYPE_F32)
     silu_mul_kernel<float, ACT><<<(int)blocks, threads, 0, stream>>>((const float*)gu,
-                                                                    (float*)out, T, I, gk, bias);
+                                                                    (float*)out, ldo, T, I, gk,
+                                                                    bias);
   else
     silu_mul_kernel<__nv_bfloat16, ACT><<<(int)blocks, threads, 0, stream>>>(
-        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, I, gk, bias);
+        (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ldo, T, I, gk, bias);
   return bf_launch_status();
 }
 
 BF_EXPORT int bf_silu_mul(const void* gu, void* out, int T, int I, int act_dtype,
                           cudaStream_t stream) {
-  return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream);
+  return gated_act_mul_launch<BF_ACT_SILU>(gu, out, I, T, I, act_dtype, stream);
 }
 
 // out[t, c] = act(gu[t, c]) * gu[t, I + c] with act 0: silu, 1: gelu's tanh form; 2: the clamped
-// form with its three constants (see BF_ACT_CLAMPED); bias: null, or 2 I numbers added to gu first.
-BF_EXPORT int bf_gated_act_mul(const void* gu, void* out, int T, int I, int act, int act_dtype,
+// form with its three constants (see BF_ACT_CLAMPED); ldo: elements between the rows of out; bias: null, or 2 I numbers added to gu first.
+BF_EXPORT int bf_gated_act_mul(const void* gu, void* out, long long ldo, int T, int I, int act,
+                               int act_dtype,
                                float limit, float slope, float up_offset, const float* bias,
                                cudaStream_t stream) {
   const BfGateConst gk = {limit, slope, up_offset};
   if (act == BF_ACT_CLAMPED)
-    return gated_act_mul_launch<BF_ACT_CLAMPED>(gu, out, T, I, act_dtype, stream, gk, bias);
+    return gated_act_mul_launch<BF_ACT_CLAMPED>(gu, out, ldo, T, I, act_dtype, stream, gk, bias);
   if (act == BF_ACT_SILU)
-    return gated_act_mul_launch<BF_ACT_SILU>(gu, out, T, I, act_dtype, stream, gk, bias);
+    return gated_act_mul_launch<BF_ACT_SILU>(gu, out, ldo, T, I, act_dtype, stream, gk, bias);
   if (act == BF_ACT_GELU_TANH)
-    return gated_act_mul_launch<BF_ACT_GELU_TANH>(gu, out, T, I, act_dtype, stream, gk, bias);
+    return gated_act_mul_launch<BF_ACT_GELU_TANH>(gu, out, ldo, T, I, act_dtype, stream, gk, bias);
   return (int)cudaErrorInvalidValue;
 }
 

@@ -15,6 +15,21 @@
 struct BfGateConst {
   float limit, slope, up_offset;
 };
+// Outputs that belong to the experts of a mixture, `ff` neighbouring ones each and the shared
+// expert's behind them: output o of token t counts w[t, expert(o)] times (w [T, cols]; the shared
+// expert counts w[t, experts] times with `shared_gate`, else once), and the shared expert's clamped
+// activation has a limit of its own.  w null: no mixture.
+struct BfMixture {
+  const float* w;
+  int cols, experts, ff, shared_gate;
+  float shared_limit;
+};
+// the weight of output o for token t; k becomes the constants of o's activation
+__device__ __forceinline__ float bf_mix_weight(const BfMixture& m, int t, int o, BfGateConst& k) {
+  if (o < m.experts * m.ff) return m.w[(size_t)t * m.cols + o / m.ff];
+  k.limit = m.shared_limit;
+  return m.shared_gate ? m.w[(size_t)t * m.cols + m.experts] : 1.f;
+}
 template <int ACT>
 __device__ __forceinline__ float bf_gate_mul(float g, float u, const BfGateConst& k) {
   if (ACT == BF_ACT_CLAMPED) {

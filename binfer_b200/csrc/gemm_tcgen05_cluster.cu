@@ -68,6 +68,13 @@ struct ClusterGemmParams {
   __nv_bfloat16* xt;
   float* partials;
   long long ldr, ldxt;
+  // The same with a norm that takes no statistic of the row: resid[t, f] = sum + add_bias[f]
+  // (+ resid[t, f] unless `assign`); xt[t, f] = bf16(tanh(alpha resid) * norm_w[f] + norm_b[f]),
+  // which is the norm's whole output.
+  const float* add_bias;        // null: none
+  const float* norm_b;          // null: none
+  float alpha;
+  int assign;
   // Fused "head norms, rotation and store into the pages" epilogue of the q/k/v projection
   // (q_out != null): a tile's columns are whole heads (bn a multiple of d) and the tile's
   // rows are shared out by token, token t to CTA t % cluster, so that an owner holds whole
@@ -95,6 +102,7 @@ struct ClusterGemmParams {
   int inter;
   BfGateConst gk;
   const float* gate_bias;       // [2 inter], added to f g and f u before the activation; or null
+  BfMixture mix;                // the outputs are a mixture's experts (ff a multiple of 8)
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -183,7 +191,8 @@ __device__ __forceinline__ void load_weights(const ClusterGemmParams& p, const C
 }
 // The epilogue's form is a template parameter, so that each instance carries only its own
 // code: with all of them behind run-time tests the plain product was 3 % slower.
-enum { FORM_PLAIN = 0, FORM_ADD_NORM = 1, FORM_QKV = 2, FORM_SWIGLU = 3, FORM_CLAMPED = 4 };
+enum { FORM_PLAIN = 0, FORM_ADD_NORM = 1, FORM_QKV = 2, FORM_SWIGLU = 3, FORM_CLAMPED = 4,
+       FORM_ADD_TANH = 5 };
 
 constexpr int CL_THREADS = 256;       // eight warps: the roles of warps 1 to 3, then the epilogue
 
@@ -193,7 +202,8 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
                     const __grid_constant__ CUtensorMap map_w, OutT* __restrict__ out,
                     const ClusterGemmParams p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  constexpr bool kNorm = FORM == FORM_ADD_NORM, kQkv = FORM == FORM_QKV, kAct = FORM == FORM_SWIGLU || FORM == FORM_CLAMPED;
+  constexpr bool kTanh = FORM == FORM_ADD_TANH;
+  constexpr bool kNorm = FORM == FORM_ADD_NORM || kTanh, kQkv = FORM == FORM_QKV, kAct = FORM == FORM_SWIGLU || FORM == FORM_CLAMPED;
   constexpr int kGate = FORM == FORM_CLAMPED ? BF_ACT_CLAMPED : BF_ACT_SILU;
   BF_TRACE_POINT(10 * BF_TR_GEMM);
   bf_pdl_trigger();
@@ -398,12 +408,21 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
               u[j] = __float_as_uint(__uint_as_float(u[j]) + __ldg(p.gate_bias + p.inter + o0 + j));
             }
         }
+        // (eight neighbouring outputs belong to one expert of a mixture)
+        BfGateConst k[2] = {p.gk, p.gk};
+        float wgt[2] = {1.f, 1.f};
+        if (p.mix.w) {
+          wgt[0] = bf_mix_weight(p.mix, row, o0, k[0]);
+          wgt[1] = bf_mix_weight(p.mix, row, o0 + 8, k[1]);
+        }
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          const float a = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j]),
-                                                  __uint_as_float(u[2 * j]), p.gk);
-          const float b = bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j + 1]),
-                                                  __uint_as_float(u[2 * j + 1]), p.gk);
+          const float a = wgt[j >> 2] * bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j]),
+                                                                __uint_as_float(u[2 * j]),
+                                                                k[j >> 2]);
+          const float b = wgt[j >> 2] * bf_gate_mul_fast<kGate>(__uint_as_float(g[2 * j + 1]),
+                                                                __uint_as_float(u[2 * j + 1]),
+                                                                k[j >> 2]);
           packed[j] = pack_bf16x2(__float_as_uint(a), __float_as_uint(b));
         }
         __nv_bfloat16* dst = p.act_out + (size_t)row * p.ldact + o0;
@@ -479,14 +498,17 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
   const int groups = slice / 4;
   const int n_plain = kQkv || kAct ? 0 : p.tokens * groups;
   float pre_r[4] = {0.f, 0.f, 0.f, 0.f}, pre_w[4] = {0.f, 0.f, 0.f, 0.f};
+  float pre_s[4] = {0.f, 0.f, 0.f, 0.f};
   if (kNorm && (int)threadIdx.x < n_plain) {
     const int g = threadIdx.x / p.tokens, t = threadIdx.x - g * p.tokens;
     const int f = tile * p.bn + rank * slice + g * 4;
 #pragma unroll
     for (int k = 0; k < 4; ++k)
       if (f + k < p.features) {
-        pre_r[k] = p.resid[(size_t)t * p.ldr + f + k];
+        pre_r[k] = kTanh && p.assign ? 0.f : p.resid[(size_t)t * p.ldr + f + k];
         pre_w[k] = p.norm_w[f + k];
+        if (kTanh && p.add_bias) pre_r[k] += p.add_bias[f + k];
+        if (kTanh && p.norm_b) pre_s[k] = p.norm_b[f + k];
       }
   }
 
@@ -593,6 +615,18 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
         float x = 0.f;
         if (f + k < p.features) {
           float* rp = p.resid + (size_t)t * p.ldr + f + k;
+          if (kTanh) {
+            float add = pre_r[k], w = pre_w[k], s = pre_s[k];
+            if (!first) {
+              add = (p.assign ? 0.f : *rp) + (p.add_bias ? p.add_bias[f + k] : 0.f);
+              w = p.norm_w[f + k];
+              s = p.norm_b ? p.norm_b[f + k] : 0.f;
+            }
+            x = add + sum[k];
+            *rp = x;
+            p.xt[(size_t)t * p.ldxt + f + k] = __float2bfloat16_rn(tanhf(p.alpha * x) * w + s);
+            continue;
+          }
           x = (first ? pre_r[k] : *rp) + sum[k];
           *rp = x;
           p.xt[(size_t)t * p.ldxt + f + k] =
@@ -601,11 +635,11 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap map_x,
         sq[k] = x * x;
       }
       // rank 0's part of recv, which this thread has read: now the squares
-      *reinterpret_cast<float4*>(recv + (g * p.tok_rows + t) * 4) =
+      if (!kTanh) *reinterpret_cast<float4*>(recv + (g * p.tok_rows + t) * 4) =
           make_float4(sq[0], sq[1], sq[2], sq[3]);
     }
   }
-  if (kNorm) {
+  if (kNorm && !kTanh) {
     // one partial sum of squares per token and CTA, its columns added in ascending order
     __syncthreads();
     for (int t = threadIdx.x; t < p.tokens; t += blockDim.x) {
@@ -819,6 +853,42 @@ BF_EXPORT int bf_gemm_bf16_cluster_add_norm(const void* x, const void* w, int to
                                                      stream);
 }
 
+// The same with a norm that takes no statistic of the row, whose output is therefore complete:
+//   resid[tokens, features] (float) = x * w^T + add_bias (+ resid unless `assign`);
+//   xt = bf16(tanh(alpha resid) * norm_w + norm_b).     add_bias and norm_b may be null.
+BF_EXPORT int bf_gemm_bf16_cluster_add_tanh(const void* x, const void* w, int tokens,
+                                            int features, int K, long long ldx, long long ldw,
+                                            int bn, int cluster, float* resid, long long ldr,
+                                            const float* add_bias, int assign, float alpha,
+                                            const float* norm_w, const float* norm_b, void* xt,
+                                            long long ldxt, int* err, cudaStream_t stream) {
+  if (tokens <= 0 || features <= 0) return 0;
+  if (tokens > CL_MAX_TOKENS || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) ||
+      ((uintptr_t)w & 15) || !resid || !norm_w || !xt)
+    return (int)cudaErrorInvalidValue;
+  if ((cluster != 1 && cluster != 2 && cluster != 4 && cluster != 8) || bn <= 0 || bn > 256 ||
+      bn % (16 * cluster))
+    return (int)cudaErrorInvalidValue;
+  ClusterGemmParams p = {};
+  p.tokens = tokens;
+  p.features = features;
+  p.K = K;
+  p.bn = bn;
+  p.cluster = cluster;
+  p.err = err;
+  p.resid = resid;
+  p.norm_w = norm_w;
+  p.xt = (__nv_bfloat16*)xt;
+  p.ldr = ldr;
+  p.ldxt = ldxt;
+  p.add_bias = add_bias;
+  p.norm_b = norm_b;
+  p.alpha = alpha;
+  p.assign = assign;
+  return launch_cluster<__nv_bfloat16, FORM_ADD_TANH>(x, w, (__nv_bfloat16*)nullptr, p, ldx, ldw,
+                                                     stream);
+}
+
 // How many clusters of c CTAs of this kernel can be resident at once (0 on an error).
 static int resident_clusters(int c) {
   static int known[9] = {-1, -1, -1, -1, -1, -1, -1, -1, -1};
@@ -954,14 +1024,17 @@ BF_EXPORT int bf_gemm_swiglu_plan(int inter, int K, int num_sms, int* bn_out) {
 // rows first) and f the factor of the norm before the projection (row_partials as in
 // bf_silu_mul_scaled; null: 1), as one kernel for at most 64 token rows.  bn from
 // bf_gemm_swiglu_plan.  act_kind BF_ACT_CLAMPED: the clamped activation with its three constants
-// in silu's place.  gate_bias: null, or 2 inter floats added to f g and f u.  Returns
-// cudaErrorInvalidValue for what it does not take.
+// in silu's place.  gate_bias: null, or 2 inter floats added to f g and f u.  mix_* (mix_w null:
+// none): the outputs are a mixture's experts and are multiplied by their tokens' weights
+// (gate_act.cuh, BfMixture).  Returns cudaErrorInvalidValue for what it does not take.
 BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int inter, int K,
                                   long long ldx, long long ldw, int bn, void* act,
                                   long long ldact, const float* row_partials, int row_count,
                                   int row_width, float row_eps, int* err, int act_kind,
                                   float limit, float slope, float up_offset,
-                                  const float* gate_bias, cudaStream_t stream) {
+                                  const float* gate_bias, const float* mix_w, int mix_cols,
+                                  int mix_experts, int mix_ff, int mix_shared_gate,
+                                  float mix_shared_limit, cudaStream_t stream) {
   if (tokens <= 0 || inter <= 0) return 0;
   if (act_kind != BF_ACT_SILU && act_kind != BF_ACT_CLAMPED) return (int)cudaErrorInvalidValue;
   if (tokens > CL_MAX_TOKENS || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) ||
@@ -979,6 +1052,9 @@ BF_EXPORT int bf_gemm_bf16_swiglu(const void* x, const void* w, int tokens, int 
   p.ldact = ldact;
   p.inter = inter;
   p.gate_bias = gate_bias;
+  p.mix = BfMixture{mix_w, mix_cols, mix_experts, mix_ff, mix_shared_gate, mix_shared_limit};
+  if (mix_w && (mix_ff <= 0 || mix_ff % 8 || mix_experts <= 0 || inter < mix_experts * mix_ff))
+    return (int)cudaErrorInvalidValue;
   p.rs.partials = row_partials;
   p.rs.count = row_count;
   p.rs.inv_width = row_width > 0 ? 1.f / (float)row_width : 0.f;

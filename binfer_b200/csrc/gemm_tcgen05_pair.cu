@@ -50,6 +50,7 @@ struct PairParams {
   int* err;
   BfGateConst gk;          // of the clamped activation (gated 2)
   const float* gate_bias;  // gated: [2 features], added to the sums before the activation; or null
+  BfMixture mix;           // gated: the outputs are a mixture's experts (ff a multiple of 32)
 };
 
 constexpr int PM = 256;                      // token rows per tile (128 per CTA)
@@ -341,10 +342,15 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
                 tmem_ld32(taddr + col, r);
                 tmem_ld32(taddr + col + 64, up);
                 pair_gate_bias<32>(r, up, tf * 128 + slab * 64 + hs * 32, p);
+                BfGateConst k = p.gk;
+                float wgt = 1.f;
+                if (p.mix.w)                 // (32 neighbouring outputs belong to one expert)
+                  wgt = bf_mix_weight(p.mix, min(t, p.tokens - 1),
+                                      tf * 128 + slab * 64 + hs * 32, k);
 #pragma unroll
                 for (int j = 0; j < 32; ++j)
-                  r[j] = __float_as_uint(pair_gate(__uint_as_float(r[j]), __uint_as_float(up[j]),
-                                                   p.gated, p.gk));
+                  r[j] = __float_as_uint(
+                      wgt * pair_gate(__uint_as_float(r[j]), __uint_as_float(up[j]), p.gated, k));
               }
 #pragma unroll
               for (int q = 0; q < 4; ++q) {
@@ -398,10 +404,12 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
               const int o0 = tf * (p.bn >> 1) + half * q + c0;
               if (t < p.tokens && o0 < p.features) {
                 pair_gate_bias<16>(g, up, o0, p);
+                BfGateConst k = p.gk;
+                const float wgt = p.mix.w ? bf_mix_weight(p.mix, t, o0, k) : 1.f;
 #pragma unroll
                 for (int j = 0; j < 16; ++j)
-                  g[j] = __float_as_uint(pair_gate(__uint_as_float(g[j]), __uint_as_float(up[j]),
-                                                   p.gated, p.gk));
+                  g[j] = __float_as_uint(
+                      wgt * pair_gate(__uint_as_float(g[j]), __uint_as_float(up[j]), p.gated, k));
                 pair_store16(out + (size_t)t * p.ldo + o0, g, vec_ok, p.features - o0, false);
               }
             }
@@ -542,7 +550,8 @@ BF_EXPORT int bf_gemm_pair_choose_bn(int tokens, int columns, int step, int num_
 // pairs of CTAs.  gated != 0: w is [2 features, K] (gate rows first) and out[t, o] =
 // silu(x . w[o]) * (x . w[features + o]), bf16 only; gated == 2: the clamped activation of
 // gate_act.cuh with its three constants instead; gate_bias ([2 features] floats, or null) is added
-// before the activation.  out_dtype: BF_DTYPE_BF16 or
+// before the activation; mix_* (mix_w null: none): the outputs are a mixture's experts and are
+// multiplied by their tokens' weights (gate_act.cuh, BfMixture).  out_dtype: BF_DTYPE_BF16 or
 // BF_DTYPE_F32.  accumulate != 0 (float out only): out += the product.  bn: accumulator
 // columns per tile (0: chosen here).  Returns
 // cudaErrorInvalidValue for shapes it does not take.
@@ -550,7 +559,9 @@ BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tok
                                 int K, long long ldx, long long ldw, long long ldo, int out_dtype,
                                 int gated, int accumulate, int bn, int num_sms, int* err,
                                 float limit, float slope, float up_offset,
-                                const float* gate_bias, cudaStream_t stream) {
+                                const float* gate_bias, const float* mix_w, int mix_cols,
+                                int mix_experts, int mix_ff, int mix_shared_gate,
+                                float mix_shared_limit, cudaStream_t stream) {
   if (tokens <= 0 || features <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || num_sms < 2)
     return (int)cudaErrorInvalidValue;
@@ -570,6 +581,10 @@ BF_EXPORT int bf_gemm_bf16_pair(const void* x, const void* w, void* out, int tok
   p.gated = gated == 2 ? 2 : (gated ? 1 : 0);
   p.gk = BfGateConst{limit, slope, up_offset};
   p.gate_bias = gated ? gate_bias : nullptr;
+  p.mix = BfMixture{gated ? mix_w : nullptr, mix_cols, mix_experts, mix_ff, mix_shared_gate,
+                    mix_shared_limit};
+  if (p.mix.w && (mix_ff <= 0 || mix_ff % 32 || mix_experts <= 0 || features < mix_experts * mix_ff))
+    return (int)cudaErrorInvalidValue;
   p.accumulate = accumulate ? 1 : 0;
   p.tiles_t = (tokens + PM - 1) / PM;
   p.tiles_f = (columns + bn - 1) / bn;

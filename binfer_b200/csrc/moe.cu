@@ -304,8 +304,8 @@ BF_EXPORT int bf_moe_route(const void* h, long long stride, const float* w, int 
 
 template <typename A, int ACT>
 __global__ void moe_act_kernel(const A* __restrict__ gu, const float* __restrict__ route_w,
-                               A* __restrict__ act, int T, int F, int E, int ff, int rw_cols,
-                               int shared_gate, BfGateConst gk, BfGateConst gk_sh) {
+                               A* __restrict__ act, long long lda, int T, int F, int E, int ff,
+                               int rw_cols, int shared_gate, BfGateConst gk, BfGateConst gk_sh) {
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (long long)T * F) return;
   const int t = (int)(i / F), c = (int)(i % F);
@@ -316,7 +316,7 @@ __global__ void moe_act_kernel(const A* __restrict__ gu, const float* __restrict
     const float g = bf_ld(gu + (size_t)t * 2 * F + c), u = bf_ld(gu + (size_t)t * 2 * F + F + c);
     r = bf_gate_mul<ACT>(g, u, e < E ? gk : gk_sh) * wgt;
   }
-  bf_st(act + i, r);
+  bf_st(act + (size_t)t * lda + c, r);
 }
 
 // bfloat16 with F, ff and the experts' total a multiple of 8: eight columns a thread (they
@@ -324,9 +324,9 @@ __global__ void moe_act_kernel(const A* __restrict__ gu, const float* __restrict
 template <int ACT>
 __global__ void moe_act_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
                                         const float* __restrict__ route_w,
-                                        __nv_bfloat16* __restrict__ act, int T, int F, int E,
-                                        int ff, int rw_cols, int shared_gate, BfGateConst gk,
-                                        BfGateConst gk_sh) {
+                                        __nv_bfloat16* __restrict__ act, long long lda, int T,
+                                        int F, int E, int ff, int rw_cols, int shared_gate,
+                                        BfGateConst gk, BfGateConst gk_sh) {
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   const int F8 = F >> 3;
   if (i >= (long long)T * F8) return;
@@ -348,47 +348,48 @@ __global__ void moe_act_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu,
                                     bf_gate_mul<ACT>(g.y, u.y, k) * wgt);
     }
   }
-  *reinterpret_cast<uint4*>(act + (size_t)t * F + c) = out;
+  *reinterpret_cast<uint4*>(act + (size_t)t * lda + c) = out;
 }
 
 // rw_cols: the columns of a row of route_w; shared_gate: column E holds the shared expert's
 // weight (else that expert's weight is one).  act_kind: BF_ACT_SILU, or BF_ACT_CLAMPED with its
-// constants (the shared expert's limit apart)
+// constants (the shared expert's limit apart).  lda: elements between the rows of act
 template <int ACT>
-static int moe_act_launch(const void* gu, const float* route_w, void* act, int T, int F, int E,
-                          int ff, int rw_cols, int shared_gate, int act_dtype, BfGateConst gk,
+static int moe_act_launch(const void* gu, const float* route_w, void* act, long long lda, int T,
+                          int F, int E, int ff, int rw_cols, int shared_gate, int act_dtype, BfGateConst gk,
                           BfGateConst gk_sh, cudaStream_t stream) {
   const long long n = (long long)T * F;
   const unsigned blocks = (unsigned)((n + 255) / 256);
-  if (act_dtype == BF_DTYPE_BF16 && F % 8 == 0 && ff % 8 == 0 &&
+  if (act_dtype == BF_DTYPE_BF16 && F % 8 == 0 && ff % 8 == 0 && lda % 8 == 0 &&
       (((uintptr_t)gu | (uintptr_t)act) & 15) == 0) {
     moe_act_bf16_vec_kernel<ACT><<<(unsigned)((n / 8 + 255) / 256), 256, 0, stream>>>(
-        (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, T, F, E, ff, rw_cols,
+        (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, lda, T, F, E, ff, rw_cols,
         shared_gate, gk, gk_sh);
     return bf_launch_status();
   }
   if (act_dtype == BF_DTYPE_F32)
     moe_act_kernel<float, ACT><<<blocks, 256, 0, stream>>>((const float*)gu, route_w, (float*)act,
-                                                           T, F, E, ff, rw_cols, shared_gate, gk,
+                                                           lda, T, F, E, ff, rw_cols, shared_gate, gk,
                                                            gk_sh);
   else
     moe_act_kernel<__nv_bfloat16, ACT><<<blocks, 256, 0, stream>>>(
-        (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, T, F, E, ff, rw_cols,
+        (const __nv_bfloat16*)gu, route_w, (__nv_bfloat16*)act, lda, T, F, E, ff, rw_cols,
         shared_gate, gk, gk_sh);
   return bf_launch_status();
 }
 
-BF_EXPORT int bf_moe_act(const void* gu, const float* route_w, void* act, int T, int F, int E,
+BF_EXPORT int bf_moe_act(const void* gu, const float* route_w, void* act, long long lda, int T,
+                         int F, int E,
                          int ff, int rw_cols, int shared_gate, int act_dtype, int act_kind,
                          float limit, float shared_limit, float slope, float up_offset,
                          cudaStream_t stream) {
   if (T <= 0 || F <= 0) return 0;
   const BfGateConst gk = {limit, slope, up_offset}, gk_sh = {shared_limit, slope, up_offset};
   if (act_kind == BF_ACT_CLAMPED)
-    return moe_act_launch<BF_ACT_CLAMPED>(gu, route_w, act, T, F, E, ff, rw_cols, shared_gate,
+    return moe_act_launch<BF_ACT_CLAMPED>(gu, route_w, act, lda, T, F, E, ff, rw_cols, shared_gate,
                                           act_dtype, gk, gk_sh, stream);
   if (act_kind == BF_ACT_SILU)
-    return moe_act_launch<BF_ACT_SILU>(gu, route_w, act, T, F, E, ff, rw_cols, shared_gate,
+    return moe_act_launch<BF_ACT_SILU>(gu, route_w, act, lda, T, F, E, ff, rw_cols, shared_gate,
                                        act_dtype, gk, gk_sh, stream);
   return (int)cudaErrorInvalidValue;
 }
@@ -585,7 +586,7 @@ __global__ void moe_sparse_down_kernel(const A* __restrict__ act, const A* __res
                                        const int* __restrict__ top_ids, A* __restrict__ out,
                                        const A* __restrict__ h, long long h_stride,
                                        const float* __restrict__ route_w, int rw_cols,
-                                       int id_col) {
+                                       int id_col, long long ldd) {
   extern __shared__ __align__(16) float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.y;
@@ -593,22 +594,22 @@ __global__ void moe_sparse_down_kernel(const A* __restrict__ act, const A* __res
   ms_stage<A>(act + (size_t)t * n_act, sh, n_act);
   __syncthreads();
   const int row0 = (blockIdx.x * MS_WARPS + warp) * MS_ROWS;
-  const bool vec = (ff % 8) == 0 && (F % 8) == 0 && (((uintptr_t)w_down) & 15) == 0;
+  const bool vec = (ff % 8) == 0 && (F % 8) == 0 && (ldd % 8) == 0 && (((uintptr_t)w_down) & 15) == 0;
   const int rows = min(MS_ROWS, width - row0);
   if (rows <= 0) return;
-  const A* wr = w_down + (size_t)row0 * F;
+  const A* wr = w_down + (size_t)row0 * ldd;       // (rows of w_down lie ldd elements apart)
   float a[MS_ROWS], part[MS_ROWS];
 #pragma unroll
   for (int r = 0; r < MS_ROWS; ++r) a[r] = 0.f;
   for (int k = 0; k < top; ++k) {
     if (top_ids[(size_t)t * top + k] >= E) continue;
-    ms_dots<A, MS_ROWS>(wr + (size_t)top_ids[(size_t)t * top + k] * ff, (size_t)F, rows,
+    ms_dots<A, MS_ROWS>(wr + (size_t)top_ids[(size_t)t * top + k] * ff, (size_t)ldd, rows,
                         sh + (size_t)k * ff, ff, lane, vec, part);
 #pragma unroll
     for (int r = 0; r < MS_ROWS; ++r) a[r] += part[r];
   }
   if (ff_sh) {
-    ms_dots<A, MS_ROWS>(wr + (size_t)E * ff, (size_t)F, rows, sh + (size_t)top * ff, ff_sh, lane,
+    ms_dots<A, MS_ROWS>(wr + (size_t)E * ff, (size_t)ldd, rows, sh + (size_t)top * ff, ff_sh, lane,
                         vec && (ff_sh % 8) == 0, part);
 #pragma unroll
     for (int r = 0; r < MS_ROWS; ++r) a[r] += part[r];
@@ -626,8 +627,8 @@ BF_EXPORT int bf_moe_sparse(const void* h, long long stride, const void* w_gu, c
                             const int* top_ids, const float* top_w, const float* route_w,
                             int rw_cols, void* act, void* out, int T, int width, int E, int ff,
                             int ff_sh, int top, int act_dtype, int shared_gate, int id_col,
-                            int act_kind, float limit, float shared_limit, float slope,
-                            float up_offset, cudaStream_t stream) {
+                            long long ldd, int act_kind, float limit, float shared_limit,
+                            float slope, float up_offset, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (act_kind != BF_ACT_SILU && act_kind != BF_ACT_CLAMPED) return (int)cudaErrorInvalidValue;
   const BfGateConst gk = {limit, slope, up_offset}, gk_sh = {shared_limit, slope, up_offset};
@@ -648,7 +649,7 @@ BF_EXPORT int bf_moe_sparse(const void* h, long long stride, const void* w_gu, c
         route_w, rw_cols, shared_gate, (float*)act, gk, gk_sh);
     moe_sparse_down_kernel<float><<<g2, MS_WARPS * 32, (size_t)n_act * 4, stream>>>(
         (const float*)act, (const float*)w_down, width, F, E, ff, ff_sh, top, top_ids,
-        (float*)out, (const float*)h, stride, route_w, rw_cols, id_col);
+        (float*)out, (const float*)h, stride, route_w, rw_cols, id_col, ldd);
   } else {
     auto k1 = act_kind == BF_ACT_CLAMPED ? moe_sparse_gate_up_kernel<__nv_bfloat16, BF_ACT_CLAMPED>
                                          : moe_sparse_gate_up_kernel<__nv_bfloat16, BF_ACT_SILU>;
@@ -657,7 +658,8 @@ BF_EXPORT int bf_moe_sparse(const void* h, long long stride, const void* w_gu, c
         top_ids, top_w, route_w, rw_cols, shared_gate, (__nv_bfloat16*)act, gk, gk_sh);
     moe_sparse_down_kernel<__nv_bfloat16><<<g2, MS_WARPS * 32, (size_t)n_act * 4, stream>>>(
         (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, width, F, E, ff, ff_sh, top,
-        top_ids, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, stride, route_w, rw_cols, id_col);
+        top_ids, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, stride, route_w, rw_cols, id_col,
+        ldd);
   }
   return bf_launch_status();
 }

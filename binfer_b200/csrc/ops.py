@@ -243,7 +243,8 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor,
     """out[t, c] = silu(f gate_up[t, c]) * f gate_up[t, I + c]; f = 1 without ``row_scale``
     (which is taken for bfloat16 and I a multiple of 8, at least 256)."""
     T, I = out.shape
-    if gate_up.shape != (T, 2 * I) or not gate_up.is_contiguous() or gate_up.dtype != out.dtype:
+    if (gate_up.shape != (T, 2 * I) or not gate_up.is_contiguous() or gate_up.dtype != out.dtype
+            or not out.is_contiguous()):
         raise KernelError("silu_mul: gate_up must be contiguous [T, 2*I] of the output's dtype")
     if row_scale is not None:
         if out.dtype != torch.bfloat16 or I % 8 or I < 256:
@@ -265,7 +266,7 @@ def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str,
     """out[t, c] = act(gate_up[t, c]) * gate_up[t, I + c]; ``activation`` one of
     ``GATE_ACTIVATIONS``.  "clamped": with g = min(gate, limit) and u = clamp(up, -limit, limit)
     the result is g sigmoid(slope g) (u + up_offset).  ``bias`` (float32 ``[2 I]``) is added to
-    the rows of ``gate_up`` first."""
+    the rows of ``gate_up`` first.  ``out`` may be a column block of a wider buffer."""
     T, I = out.shape
     if bias is not None:
         _want(bias, torch.float32, "bias")
@@ -275,7 +276,10 @@ def gated_act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str,
         raise KernelError(f"gated_act_mul: unknown activation {activation!r}")
     if gate_up.shape != (T, 2 * I) or not gate_up.is_contiguous() or gate_up.dtype != out.dtype:
         raise KernelError("gated_act_mul: gate_up must be contiguous [T, 2*I] of the output's dtype")
-    _run("gated_act_mul", lib().bf_gated_act_mul, _ptr(gate_up), _ptr(out), _c_int(T), _c_int(I),
+    if out.stride(1) != 1:
+        raise KernelError("gated_act_mul: rows of out must be contiguous")
+    _run("gated_act_mul", lib().bf_gated_act_mul, _ptr(gate_up), _ptr(out), _c_ll(out.stride(0)),
+         _c_int(T), _c_int(I),
          _c_int(GATE_ACTIVATIONS[activation]), _c_int(_dtype_code(out)), _c_float(limit),
          _c_float(slope), _c_float(up_offset), _ptr(bias), _stream())
 
@@ -1109,15 +1113,17 @@ def moe_act(gu: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor, experts:
     ``expert(c) = c // ff`` for ``c < experts * ff``; the columns behind the experts' (a shared
     expert) take column ``experts`` of ``route_w`` when ``shared_gate``, else the weight one
     (None: when ``route_w`` has exactly one column more than there are experts).
-    ``expert_act``: another activation in silu's place."""
+    ``expert_act``: another activation in silu's place.  ``act`` may be a column block of a wider
+    buffer."""
     T, F = act.shape
     _want(route_w, torch.float32, "route_w")
-    if tuple(gu.shape) != (T, 2 * F) or not gu.is_contiguous() or not act.is_contiguous() \
+    if tuple(gu.shape) != (T, 2 * F) or not gu.is_contiguous() or act.stride(1) != 1 \
             or gu.dtype != act.dtype or route_w.shape[0] != T or not route_w.is_contiguous():
         raise KernelError("moe_act: gu must be contiguous [T, 2 F] of act's type")
     if shared_gate is None:
         shared_gate = route_w.shape[1] == experts + 1
-    _run("moe_act", lib().bf_moe_act, _ptr(gu), _ptr(route_w), _ptr(act), _c_int(T), _c_int(F),
+    _run("moe_act", lib().bf_moe_act, _ptr(gu), _ptr(route_w), _ptr(act),
+         _c_ll(act.stride(0)), _c_int(T), _c_int(F),
          _c_int(experts), _c_int(ff), _c_int(route_w.shape[1]), _c_int(1 if shared_gate else 0),
          _c_int(_dtype_code(act)), *expert_act.args(), _stream())
 
@@ -1158,7 +1164,7 @@ def moe_sparse(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
     if shared_gate is None:
         shared_gate = route_w.shape[1] == experts + 1
     if (tuple(w_gate_up.shape) != (2 * F, width) or tuple(w_down.shape) != (width, F)
-            or not w_gate_up.is_contiguous() or not w_down.is_contiguous()
+            or not w_gate_up.is_contiguous() or w_down.stride(1) != 1
             or w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or h.stride(1) != 1
             or not out.is_contiguous() or out.dtype != h.dtype):
         raise KernelError("moe_sparse: stacked weights [2 F, width] and [width, F] of h's type")
@@ -1171,7 +1177,7 @@ def moe_sparse(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
          _ptr(w_down), _ptr(top_ids), _ptr(top_w), _ptr(route_w), _c_int(route_w.shape[1]),
          _ptr(act), _ptr(out), _c_int(T), _c_int(width), _c_int(experts), _c_int(ff),
          _c_int(ff_sh), _c_int(top), _c_int(_dtype_code(h)), _c_int(1 if shared_gate else 0),
-         _c_int(identity_col), *expert_act.args(), _stream())
+         _c_int(identity_col), _c_ll(w_down.stride(0)), *expert_act.args(), _stream())
     global _launches
     _launches += 1          # two kernels
 
@@ -1716,12 +1722,14 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Te
 def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: torch.Tensor,
                    bn: int = 0, gated: bool = False, accumulate: bool = False,
                    activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
-                   up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None) -> bool:
+                   up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None,
+                   mixture: Optional["Mixture"] = None) -> bool:
     """out[M, N] = x[M, K] @ w[N, K]^T on pairs of SMs (``tcgen05.mma.cta_group::2``, tiles of
     256 token rows): the product for many token rows.  ``gated``: ``w`` is the stacked
     ``[2 N, K]`` gate/up weight and ``out[M, N] = silu(x w_gate^T) * (x w_up^T)``, bfloat16
     only; ``activation`` "clamped" with its constants as in ``gated_act_mul`` in silu's place.
-    ``gate_bias`` (float32 ``[2 N]``) is added to the sums before the activation.
+    ``gate_bias`` (float32 ``[2 N]``) is added to the sums before the activation.  ``mixture``: the
+    outputs are multiplied by their tokens' weights for the experts that they belong to.
     ``accumulate``: ``out`` (float32) ``+=`` the product.  ``bn``: accumulator columns
     per tile (0: chosen by the library).  Returns False, having done nothing, for shapes the
     kernel does not take."""
@@ -1744,8 +1752,34 @@ def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: tor
          _c_int(_dtype_code(out)),
          _c_int((2 if activation == "clamped" else 1) if gated else 0),
          _c_int(1 if accumulate else 0), _c_int(bn), _c_int(num_sms(x.device)), _ptr(err),
-         _c_float(limit), _c_float(slope), _c_float(up_offset), _gate_bias(gate_bias, w), _stream())
+         _c_float(limit), _c_float(slope), _c_float(up_offset), _gate_bias(gate_bias, w),
+         *_mixture_args(mixture, M, N, 32), _stream())
     return True
+
+
+class Mixture:
+    """The outputs of a gated product as the experts of a mixture: ``ff`` neighbouring outputs per
+    expert and the shared expert's behind them, each multiplied by the token's weight for it,
+    ``route_w [T, cols]`` (column ``experts`` is the shared expert's with ``shared_gate``, else it
+    counts once); the shared expert's clamped activation has the limit ``shared_limit``."""
+    __slots__ = ("route_w", "experts", "ff", "shared_gate", "shared_limit")
+
+    def __init__(self, route_w: torch.Tensor, experts: int, ff: int, shared_gate: bool,
+                 shared_limit: float = 0.0):
+        _want(route_w, torch.float32, "route_w")
+        self.route_w, self.experts, self.ff = route_w, experts, ff
+        self.shared_gate, self.shared_limit = shared_gate, shared_limit
+
+
+def _mixture_args(m: Optional[Mixture], T: int, outputs: int, step: int):
+    if m is None:
+        return (_ptr(None), _c_int(0), _c_int(0), _c_int(0), _c_int(0), _c_float(0.0))
+    if (m.ff <= 0 or m.ff % step or outputs < m.experts * m.ff or m.route_w.shape[0] != T
+            or m.route_w.shape[1] < m.experts + (1 if m.shared_gate else 0)):
+        raise KernelError(f"gated product: a mixture's experts need a multiple of {step} outputs "
+                          f"each, and a row of weights per token")
+    return (_ptr(m.route_w), _c_int(m.route_w.shape[1]), _c_int(m.experts), _c_int(m.ff),
+            _c_int(1 if m.shared_gate else 0), _c_float(m.shared_limit))
 
 
 def _gate_bias(bias: Optional[torch.Tensor], w: torch.Tensor):
@@ -1814,6 +1848,34 @@ def gemm_bf16_cluster_add_norm(x: torch.Tensor, w: torch.Tensor, resid: torch.Te
     return xt, RowScale(partials, N, eps)
 
 
+def gemm_bf16_cluster_add_tanh(x: torch.Tensor, w: torch.Tensor, resid: torch.Tensor,
+                               bias: Optional[torch.Tensor], alpha: float, norm_w: torch.Tensor,
+                               norm_b: Optional[torch.Tensor], err: torch.Tensor, bn: int,
+                               cluster: int, assign: bool = False) -> Optional[torch.Tensor]:
+    """``resid += x @ w^T + bias`` (``assign``: ``=``; float32 stream ``[M, N]``), and the output
+    of the next norm, ``bfloat16(tanh(alpha resid) * norm_w + norm_b)``, which is returned, or
+    None, having done nothing, for shapes the kernel does not take (M <= 64, see
+    ``gemm_bf16_cluster``)."""
+    M, K = x.shape
+    N = w.shape[0]
+    if (M > CLUSTER_MAX_TOKENS or K % 8 or x.stride(1) != 1 or w.stride(1) != 1 or x.stride(0) % 8
+            or w.stride(0) % 8 or x.data_ptr() % 16 or w.data_ptr() % 16
+            or resid.dtype != torch.float32 or resid.shape != (M, N) or resid.stride(1) != 1):
+        return None
+    for name, t in (("bias", bias), ("norm_w", norm_w), ("norm_b", norm_b)):
+        if t is not None:
+            _want(t, torch.float32, name)
+            if t.numel() != N:
+                raise KernelError(f"gemm_bf16_cluster_add_tanh: {name} must have N numbers")
+    xt = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+    _run("gemm_bf16_cluster_add_tanh", lib().bf_gemm_bf16_cluster_add_tanh, _ptr(x), _ptr(w),
+         _c_int(M), _c_int(N), _c_int(K), _c_ll(x.stride(0)), _c_ll(w.stride(0)), _c_int(bn),
+         _c_int(cluster), _ptr(resid), _c_ll(resid.stride(0)), _ptr(bias),
+         _c_int(1 if assign else 0), _c_float(alpha), _ptr(norm_w), _ptr(norm_b), _ptr(xt),
+         _c_ll(xt.stride(0)), _ptr(err), _stream())
+    return xt
+
+
 def num_sms(device: torch.device) -> int:
     sms = _num_sms.get(device.index)
     if sms is None:
@@ -1878,7 +1940,8 @@ def gemm_swiglu_plan(inter: int, K: int, device: torch.device):
 def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor,
                      err: torch.Tensor, bn: int, row_scale: Optional[RowScale] = None,
                      activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
-                     up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None) -> bool:
+                     up_offset: float = 0.0, gate_bias: Optional[torch.Tensor] = None,
+                     mixture: Optional["Mixture"] = None) -> bool:
     """``silu_mul(x @ w_gate_up^T)`` as one kernel for at most 64 token rows: ``w_gate_up`` is
     ``[2 I, K]`` with the gate rows first, ``out`` is ``[M, I]``.  ``activation`` "clamped" with its
     constants as in ``gated_act_mul`` in silu's place.  Returns False, having done
@@ -1897,7 +1960,8 @@ def gemm_bf16_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor
          _c_int(I), _c_int(K), _c_ll(x.stride(0)), _c_ll(w_gate_up.stride(0)), _c_int(bn),
          _ptr(out), _c_ll(out.stride(0)), *_row_scale_args(row_scale, M), _ptr(err),
          _c_int(GATE_ACTIVATIONS[activation]), _c_float(limit), _c_float(slope),
-         _c_float(up_offset), _gate_bias(gate_bias, w_gate_up), _stream())
+         _c_float(up_offset), _gate_bias(gate_bias, w_gate_up), *_mixture_args(mixture, M, I, 8),
+         _stream())
     return True
 
 

@@ -35,7 +35,8 @@ from ..cache.manager import KVNeed, StateNeed
 from ..config.specs import ConvWindowAttentionSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .base import BuildEnv, EntryView, Mixer, StepContext, build_position, register_mixer
+from .base import (BuildEnv, EntryView, Mixer, StackedOut, StepContext, build_position,
+                   register_mixer)
 from .linear import linear
 
 # BINFER_B200_CWA_TENSOR_CORES=0: the one-warp-per-row kernel also in bfloat16 (the float32
@@ -49,7 +50,7 @@ DECODE_KERNEL = os.environ.get("BINFER_B200_CWA_DECODE_KERNEL", "1") != "0"
 PREFILL_KERNEL_ROWS = 256
 
 
-class ConvWindowAttention(Mixer):
+class ConvWindowAttention(Mixer, StackedOut):
     def __init__(self, spec: ConvWindowAttentionSpec, hidden_size: int, prefix: str,
                  env: BuildEnv):
         if spec.num_heads % spec.num_kv_heads:
@@ -172,6 +173,11 @@ class ConvWindowAttention(Mixer):
         out = torch.empty((x.shape[0], self.out_cols), dtype=x.dtype, device=x.device)
         self.run(linear(x, self.w_in), ctx, view, out, 1.0)
         return linear(out, self.w_out)
+
+    def forward_inner(self, x: torch.Tensor, ctx: StepContext, view: EntryView,
+                      out: torch.Tensor) -> bool:
+        self.run(linear(x, self.w_in), ctx, view, out, 1.0)
+        return True
 
     def run(self, proj: torch.Tensor, ctx: StepContext, view: EntryView, out: torch.Tensor,
             out_scale: float) -> None:

@@ -32,7 +32,8 @@ from ..cache.manager import KVNeed
 from ..config.specs import LatentAttentionSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .base import BuildEnv, EntryView, Mixer, StepContext, build_position, register_mixer
+from .base import (BuildEnv, EntryView, Mixer, StackedOut, StepContext, build_position,
+                   register_mixer)
 from .linear import linear, linear_heads
 
 # BINFER_B200_LATENT_TENSOR_CORES=0: the one-warp-per-row kernel also in bfloat16 (the float32
@@ -40,7 +41,7 @@ from .linear import linear, linear_heads
 TENSOR_CORES = os.environ.get("BINFER_B200_LATENT_TENSOR_CORES", "1") != "0"
 
 
-class LatentAttention(Mixer):
+class LatentAttention(Mixer, StackedOut):
     def __init__(self, spec: LatentAttentionSpec, hidden_size: int, prefix: str, env: BuildEnv):
         s = spec
         if min(s.num_heads, s.head_dim, s.value_dim, s.kv_rank) <= 0 or s.rot_dim < 0:
@@ -66,7 +67,8 @@ class LatentAttention(Mixer):
                 raise ValueError("latent attention takes rotary encodings only")
         self.names = dict(s.names)
         self.gate_off = self.q_rows + self.kv_size
-        self.w_proj = self.w_ukT = self.w_uv = self.w_o = self.norm_w = None
+        self.out_cols = self.H * self.dv
+        self.w_proj = self.w_ukT = self.w_uv = self.w_out = self.norm_w = None
         self.w_uq = self.q_norm_w = self.sinks = None
 
     # ----------------------------------------------------------------- weights
@@ -104,7 +106,7 @@ class LatentAttention(Mixer):
         # [dv, rank] expands a mixture of latents into the head's value
         self.w_ukT = g("uk").view(self.H, self.d, self.rank).transpose(1, 2).contiguous()
         self.w_uv = g("uv").view(self.H, self.dv, self.rank).contiguous()
-        self.w_o = g("o")
+        self.w_out = g("o")
         if self.spec.sinks:
             self.sinks = g("sink")
 
@@ -114,6 +116,14 @@ class LatentAttention(Mixer):
 
     # ----------------------------------------------------------------- forward
     def forward(self, x: torch.Tensor, ctx: StepContext, view: EntryView) -> torch.Tensor:
+        out = torch.empty((x.shape[0], self.out_cols), dtype=x.dtype, device=x.device)
+        self.forward_inner(x, ctx, view, out)
+        return linear(out, self.w_out)
+
+    def forward_inner(self, x: torch.Tensor, ctx: StepContext, view: EntryView,
+                      out: torch.Tensor) -> bool:
+        """Everything but the output projection, into ``out [T, heads * value_dim]`` (which may be
+        a column block of a wider buffer)."""
         s, T, H = self.spec, x.shape[0], self.H
         if not view.writes_cache:
             raise ValueError("latent attention keeps a cache of its own")
@@ -150,12 +160,18 @@ class LatentAttention(Mixer):
                 ctx.positions, ctx.block_tables[g], o_lat.view(T, H * self.rank), H, 1,
                 self.kv_size, None, s.softmax_scale, ctx.err, value_dim=self.rank,
                 v_stride=self.kv_size, sinks=self.sinks)
-        out = torch.empty((T, H, self.dv), dtype=x.dtype, device=x.device)
-        linear_heads(o_lat, self.w_uv, out)
-        out = out.view(T, H * self.dv)
-        if s.head_gate:
-            ops.head_gate_mul(out, proj[:, self.gate_off:self.gate_off + H], H, self.dv)
-        return linear(out, self.w_o)
+        heads = out.unflatten(1, (H, self.dv))
+        if not s.head_gate or out.is_contiguous():
+            linear_heads(o_lat, self.w_uv, heads)
+            if s.head_gate:
+                ops.head_gate_mul(out, proj[:, self.gate_off:self.gate_off + H], H, self.dv)
+            return True
+        own = torch.empty((T, H, self.dv), dtype=x.dtype, device=x.device)
+        linear_heads(o_lat, self.w_uv, own)
+        own = own.view(T, H * self.dv)
+        ops.head_gate_mul(own, proj[:, self.gate_off:self.gate_off + H], H, self.dv)
+        out.copy_(own)
+        return True
 
 
 register_mixer("latent_attention", LatentAttention)

@@ -182,6 +182,25 @@ class DeferredLinear:
         return y
 
 
+class StackedOut:
+    """Interface of a part whose last step is a product (optional): what lies in front of it can be
+    written into a column block of a buffer that the part shares with another one, so that one
+    product against both weights side by side makes the sum of the two parts' outputs.
+
+    ``w_out [hidden, out_cols]`` is the product's weight (the block may put a column block of a
+    stacked weight in its place), ``out_bias`` a float32 vector or None; ``forward_inner`` writes
+    ``[T, out_cols]`` into ``out`` and returns True, or returns False, having done nothing, where
+    this step has a way of its own."""
+
+    out_cols: int
+    w_out: Optional[torch.Tensor] = None
+    out_bias: Optional[torch.Tensor] = None
+
+    def forward_inner(self, x: torch.Tensor, ctx: StepContext, view: Optional["EntryView"],
+                      out: torch.Tensor) -> bool:
+        raise NotImplementedError
+
+
 class ScaledRows:
     """Activations ``[T, H]`` whose rows still lack a common factor (``scale``, an
     ``ops.RowScale``): a norm's output as a fused product leaves it.  A part that sets
@@ -278,9 +297,16 @@ class ResidualStream:
         ``consumer`` the part that takes its output; the fused path needs a norm with a
         ``fused_scale`` (weight, eps) over whole rows and a consumer that accepts
         :class:`ScaledRows`."""
-        from .linear import linear_add_norm
+        from .linear import linear, linear_add_norm
         fs = getattr(norm, "fused_scale", None)
         self.reading = None
+        whole = getattr(norm, "fused_add_linear", None)
+        if whole is not None:          # a norm whose output the product's epilogue can finish
+            self.flush()
+            out = whole(self.x, d)
+            if out is not None:
+                self.ready, self.ready_for = out, norm
+                return
         if (fs is not None and getattr(consumer, "accepts_scaled_rows", False)
                 and d.bias is None):
             self.flush()
@@ -289,7 +315,23 @@ class ResidualStream:
             if got is not None:
                 self.ready, self.ready_for = ScaledRows(*got), norm
                 return
-        self.add(d.compute())
+        self.add(linear(d.x, d.w), d.bias)
+
+    def replace_linear(self, d: DeferredLinear, norm=None) -> None:
+        """The stream becomes ``d.x @ d.w^T`` (what it was, and its pending adds, are in
+        ``d.x``); ``norm`` is the norm that reads it next."""
+        from .linear import linear
+        self.replace(self.x)
+        whole = getattr(norm, "fused_add_linear", None)
+        if whole is not None:
+            out = whole(self.x, d, assign=True)
+            if out is not None:
+                self.ready, self.ready_for = out, norm
+                return
+        self.replace(linear(d.x, d.w, out_dtype=torch.float32))
+        if d.bias is not None:
+            from ..csrc import ops
+            ops.bias_add(self.x, d.bias)
 
     def flush(self) -> None:
         from ..csrc import ops

@@ -191,6 +191,24 @@ def linear_add_norm(x: torch.Tensor, w: torch.Tensor, resid: torch.Tensor,
                                           *plan)
 
 
+def linear_add_tanh(x: torch.Tensor, w: torch.Tensor, resid: torch.Tensor,
+                    bias: Optional[torch.Tensor], alpha: float, norm_w: torch.Tensor,
+                    norm_b: Optional[torch.Tensor], assign: bool = False):
+    """``resid += x @ w^T + bias`` (``assign``: ``=``) with the next norm, ``tanh(alpha resid) *
+    norm_w + norm_b``, in the same kernel: returns the norm's output, or None, having done
+    nothing, where the cluster kernel does not run."""
+    M, (N, K) = x.shape[0], w.shape
+    if (not FUSE_NORM or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16
+            or not _use_cluster(M, N, K)):
+        return None
+    plan = _plans.get((N, K))
+    if plan is None:
+        plan = _plans[(N, K)] = ops.gemm_cluster_plan(N, K, x.device) or False
+    if not plan:
+        return None
+    return ops.gemm_bf16_cluster_add_tanh(x, w, resid, bias, alpha, norm_w, norm_b,
+                                          ops.error_word(x.device), *plan, assign=assign)
+
 
 def linear_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """``out[:, h] = x[:, h] @ w[h]^T`` for every head h: ``x [T, H, K]`` and ``out [T, H, N]``

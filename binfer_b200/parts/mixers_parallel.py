@@ -22,11 +22,12 @@ import torch
 from ..cache.manager import KVNeed, StateNeed
 from ..config.specs import ParallelMixersSpec
 from ..weights.loader import ParamSpec
-from .base import BuildEnv, EntryView, Mixer, StepContext, build_mixer, register_mixer
+from .base import (BuildEnv, EntryView, Mixer, StackedOut, StepContext, build_mixer,
+                   register_mixer)
 from .linear import linear
 
 
-class ParallelMixers(Mixer):
+class ParallelMixers(Mixer, StackedOut):
     def __init__(self, spec: ParallelMixersSpec, hidden_size: int, prefix: str, env: BuildEnv):
         if not spec.branches:
             raise ValueError("parallel mixers need at least one branch")
@@ -86,15 +87,19 @@ class ParallelMixers(Mixer):
         return StateNeed((self.state_size,), "float32") if self.state_size else None
 
     def forward(self, x: torch.Tensor, ctx: StepContext, view: EntryView) -> torch.Tensor:
-        T = x.shape[0]
+        acts = torch.empty((x.shape[0], self.out_cols), dtype=x.dtype, device=x.device)
+        self.forward_inner(x, ctx, view, acts)
+        return linear(acts, self.w_out)
+
+    def forward_inner(self, x: torch.Tensor, ctx: StepContext, view: EntryView,
+                      acts: torch.Tensor) -> bool:
         proj = linear(x, self.w_in)
-        acts = torch.empty((T, self.out_cols), dtype=x.dtype, device=x.device)
         for m, scale, a, b, (so, sn) in zip(self.branches, self.scales, self.in_off, self.out_off,
                                             self.state_cols):
             sub = dataclasses.replace(
                 view, state=view.state[:, so:so + sn] if sn else None)
             m.run(proj[:, a:a + m.in_rows], ctx, sub, acts[:, b:b + m.out_cols], scale)
-        return linear(acts, self.w_out)
+        return True
 
 
 register_mixer("parallel_mixers", ParallelMixers)

@@ -20,8 +20,8 @@ import torch
 from ..config.specs import GatedMLPSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .base import (BuildEnv, DeferredLinear, FeedForward, ScaledRows, StepContext, register_ffn,
-                   split_scaled)
+from .base import (BuildEnv, DeferredLinear, FeedForward, ScaledRows, StackedOut, StepContext,
+                   register_ffn, split_scaled)
 from .linear import linear, pair_token_limit, swiglu_token_limit
 
 # BINFER_B200_FUSE_SWIGLU=0: the stacked gate/up projection and the activation as two kernels
@@ -30,7 +30,7 @@ FUSE_SWIGLU = os.environ.get("BINFER_B200_FUSE_SWIGLU", "1") != "0"
 FUSE_SWIGLU_FILL = 0.5
 
 
-class GatedMLP(FeedForward):
+class GatedMLP(FeedForward, StackedOut):
     def __init__(self, spec: GatedMLPSpec, hidden_size: int, prefix: str, env: BuildEnv):
         if spec.activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"activation {spec.activation!r} is not supported (supported: "
@@ -43,8 +43,9 @@ class GatedMLP(FeedForward):
             raise ValueError("a clamped activation needs a positive limit")
         self.spec, self.hidden, self.prefix, self.env = spec, hidden_size, prefix, env
         self.inter = spec.intermediate_size
-        self.w_gate_up = self.w_down = None
-        self.b_gate_up = self.b_down = None     # float32, with GatedMLPSpec.bias
+        self.out_cols = self.inter
+        self.w_gate_up = self.w_out = None
+        self.b_gate_up = self.out_bias = None   # float32, with GatedMLPSpec.bias
         self._swiglu_plan = None
 
     def param_specs(self) -> List[ParamSpec]:
@@ -62,10 +63,10 @@ class GatedMLP(FeedForward):
     def load(self, get: Callable[[ParamSpec], torch.Tensor]) -> None:
         g, u, d, *biases = self.param_specs()
         self.w_gate_up = torch.cat([get(g), get(u)], dim=0).contiguous()
-        self.w_down = get(d)
+        self.w_out = get(d)
         if biases:
             bg, bu, bd = (get(b) for b in biases)
-            self.b_gate_up, self.b_down = torch.cat([bg, bu]).contiguous(), bd
+            self.b_gate_up, self.out_bias = torch.cat([bg, bu]).contiguous(), bd
 
     accepts_scaled_rows = True
 
@@ -79,13 +80,22 @@ class GatedMLP(FeedForward):
             x = x.dense()                  # the activation kernel takes the factor at other sizes only
         x, row_scale = split_scaled(x)
         h = torch.empty((x.shape[0], self.inter), dtype=x.dtype, device=x.device)
-        if not self._project_fused(x, h, row_scale):
-            gu = linear(x, self.w_gate_up)
-            if self.silu and self.b_gate_up is None:
-                ops.silu_mul(gu, h, row_scale=row_scale)
-            else:
-                ops.gated_act_mul(gu, h, bias=self.b_gate_up, **self._act)
-        return DeferredLinear(h, self.w_down, self.b_down)
+        self._inner(x, h, row_scale)
+        return DeferredLinear(h, self.w_out, self.out_bias)
+
+    def forward_inner(self, x, ctx: StepContext, view, out: torch.Tensor) -> bool:
+        self._inner(x, out, None)
+        return True
+
+    def _inner(self, x, h, row_scale) -> None:
+        """Gate, up and activation into ``h`` (which may be a column block of a wider buffer)."""
+        if self._project_fused(x, h, row_scale):
+            return
+        gu = linear(x, self.w_gate_up)
+        if self.silu and self.b_gate_up is None and h.is_contiguous():
+            ops.silu_mul(gu, h, row_scale=row_scale)
+        else:
+            ops.gated_act_mul(gu, h, bias=self.b_gate_up, **self._act)
 
     def _project_fused(self, x, h, row_scale) -> bool:
         """Few token rows in bfloat16: the stacked projection with the activation in its

@@ -20,7 +20,8 @@ from ..cache.manager import CacheManager, KVNeed, StateNeed
 from ..config.specs import ModelSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec, TensorSource, check_names, place
-from .base import (BuildEnv, EntryView, ResidualStream, StepContext, build_block, build_norm)
+from .base import (BuildEnv, DeferredLinear, EntryView, ResidualStream, StepContext, build_block,
+                   build_norm)
 from .linear import linear
 
 # importing the modules registers the built-in parts
@@ -136,9 +137,10 @@ class DecoderModel:
         for obj in [self] + self.blocks + [self.final_norm] + \
                 [p for b in self.blocks for p in (b.parts() if hasattr(b, "parts") else [])]:
             for v in vars(obj).values():
-                if isinstance(v, torch.Tensor) and v.data_ptr() not in seen:
-                    seen.add(v.data_ptr())
-                    total += v.numel() * v.element_size()
+                # (by storage: a part's weight may be a column block of a stacked one)
+                if isinstance(v, torch.Tensor) and v.untyped_storage().data_ptr() not in seen:
+                    seen.add(v.untyped_storage().data_ptr())
+                    total += v.untyped_storage().nbytes()
         return total
 
     # ------------------------------------------------------------------- cache
@@ -186,7 +188,7 @@ class DecoderModel:
             ctx.entry = e
             block = self.blocks[entry.layer]
             if entry.before is not None:
-                self._open_pass(stream, ctx, entry.before)
+                self._open_pass(stream, ctx, entry.before, getattr(block, "first_norm", None))
             if getattr(block, "takes_successor", False):
                 # a block may let its last product prepare the next block's first norm
                 # (not where the stream changes in between: the start of a pass)
@@ -210,17 +212,17 @@ class DecoderModel:
         return logits
 
 
-    def _open_pass(self, stream: ResidualStream, ctx: StepContext, before) -> None:
+    def _open_pass(self, stream: ResidualStream, ctx: StepContext, before, norm=None) -> None:
         """Fold the pending sublayer output into the stream together with what a pass starts
         with: the embedding output again (gathered from the table anew, in float) and a row
         of the pass table; or replace the stream by the pass projection of itself and the
-        embedding output."""
+        embedding output.  ``norm``: the norm that reads the stream next, if the block says so."""
         if before.project:
             pair = torch.empty((ctx.T, 2 * self.spec.hidden_size), dtype=self.env.dtype,
                                device=self.env.device)
             ops.stream_pair(stream.x, stream.pending, stream.pending2, stream.pending_bias,
                             self.embed, ctx.token_ids, self.spec.embedding_scale, pair, ctx.err)
-            stream.replace(linear(pair, self.pass_proj, out_dtype=torch.float32))
+            stream.replace_linear(DeferredLinear(pair, self.pass_proj), norm)
             return
         if not before.embedding and before.row is None:
             return

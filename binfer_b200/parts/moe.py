@@ -6,9 +6,9 @@ for every token, times ``sigmoid(w_sg . h)`` when it has a gate.  Expert: ``W_do
 (silu(W_gate h) * (W_up h))``.
 
 How it runs here: the gate and up projections of all experts (and the shared one) are one
-stacked weight, so one product gives every expert's pre-activations; a kernel applies the
-activation and multiplies each expert's block by the token's weight for it (zero when not
-chosen); one product with the down projections laid side by side then sums the weighted
+stacked weight, so one product gives every expert's pre-activations; the activation is applied
+and each expert's block multiplied by the token's weight for it (zero when not chosen), in that
+product's epilogue where its kernels take the step, else by a kernel behind it; one product with the down projections laid side by side then sums the weighted
 experts in its own accumulation.  Unchosen experts cost arithmetic but no extra pass over
 memory, no token is moved, and a token's result does not depend on what else is in the
 batch.
@@ -39,15 +39,18 @@ import torch
 from ..config.specs import MoESpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .base import BuildEnv, FeedForward, StepContext, register_ffn
-from .linear import linear
+from .base import BuildEnv, FeedForward, StackedOut, StepContext, register_ffn
+from .linear import linear, pair_token_limit, swiglu_token_limit
+from .mlp import FUSE_SWIGLU_FILL
 
 
 # BINFER_B200_MOE_SPARSE=0: every step computes every expert
 SPARSE = os.environ.get("BINFER_B200_MOE_SPARSE", "1") != "0"
+# BINFER_B200_FUSE_EXPERTS=0: the experts' gate/up product and their activation as two kernels
+FUSE_EXPERTS = os.environ.get("BINFER_B200_FUSE_EXPERTS", "1") != "0"
 
 
-class MoEFeedForward(FeedForward):
+class MoEFeedForward(FeedForward, StackedOut):
     def __init__(self, spec: MoESpec, hidden_size: int, prefix: str, env: BuildEnv):
         if spec.activation not in ops.FUSED_ACTIVATIONS:
             raise ValueError(f"activation {spec.activation!r} is not supported (supported: "
@@ -80,7 +83,9 @@ class MoEFeedForward(FeedForward):
         # of the chosen identity outputs
         self.cols = self.E + (1 if self.gated_shared else 0) + (1 if self.identity else 0)
         self.id_col = self.cols - 1 if self.identity else -1
-        self.w_gate_up = self.w_down = self.w_router = self.correction = None
+        self.out_cols = self.F
+        self.w_gate_up = self.w_out = self.w_router = self.correction = None
+        self._gated_plan = None
 
     def _expert_specs(self, p: str, ff: int) -> List[ParamSpec]:
         gate, up, down = self.spec.names
@@ -116,13 +121,13 @@ class MoEFeedForward(FeedForward):
         groups = self._groups()
         self.w_gate_up = torch.cat([get(g[0]) for g in groups] + [get(g[1]) for g in groups],
                                    dim=0).contiguous()
-        self.w_down = torch.cat([get(g[2]) for g in groups], dim=1).contiguous()
+        self.w_out = torch.cat([get(g[2]) for g in groups], dim=1).contiguous()
         # the router (and the shared expert's gate as one more row) in float
         self.w_router = torch.cat([get(s) for s in self._router_specs()], dim=0).contiguous()
         if self.spec.correction:
             self.correction = get(self._correction_spec())
 
-    def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+    def _route(self, x: torch.Tensor):
         T, s = x.shape[0], self.spec
         route_w = torch.empty((T, self.cols), dtype=torch.float32, device=x.device)
         top_ids = torch.empty((T, self.top), dtype=torch.int32, device=x.device)
@@ -132,22 +137,66 @@ class MoEFeedForward(FeedForward):
                       groups_keep=s.groups_keep, identity=self.identity,
                       route_scale=s.route_scale, weight_eps=s.weight_eps,
                       group_top=s.group_top, normalize=s.normalize)
-        if (SPARSE and x.dtype == torch.bfloat16 and 2 * T * self.top <= self.E
-                and ops.moe_sparse_takes(self.hidden, self.ff, self.ff_sh, self.top)):
-            # so few tokens that most experts are chosen by none: read the chosen ones alone
-            out = torch.empty((T, self.hidden), dtype=x.dtype, device=x.device)
-            ops.moe_sparse(x, self.w_gate_up, self.w_down, top_ids, top_w, route_w, out, self.E,
+        return route_w, top_ids, top_w
+
+    def _sparse(self, x: torch.Tensor) -> bool:
+        """So few tokens that most experts are chosen by none."""
+        return (SPARSE and x.dtype == torch.bfloat16 and 2 * x.shape[0] * self.top <= self.E
+                and ops.moe_sparse_takes(self.hidden, self.ff, self.ff_sh, self.top))
+
+    def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        route_w, top_ids, top_w = self._route(x)
+        if self._sparse(x):
+            # read the chosen experts alone
+            out = torch.empty((x.shape[0], self.hidden), dtype=x.dtype, device=x.device)
+            ops.moe_sparse(x, self.w_gate_up, self.w_out, top_ids, top_w, route_w, out, self.E,
                            self.ff, self.ff_sh, self.top, shared_gate=self.gated_shared,
                            identity_col=self.id_col, expert_act=self.expert_act)
             return out
-        gu = linear(x, self.w_gate_up)
-        act = torch.empty((T, self.F), dtype=x.dtype, device=x.device)
-        ops.moe_act(gu, route_w, act, self.E, self.ff, shared_gate=self.gated_shared,
-                    expert_act=self.expert_act)
-        out = linear(act, self.w_down)
+        act = torch.empty((x.shape[0], self.F), dtype=x.dtype, device=x.device)
+        self._activations(x, route_w, act)
+        out = linear(act, self.w_out)
         if self.identity:
             ops.moe_identity_add(out, x, route_w, self.id_col)
         return out
+
+    def forward_inner(self, x: torch.Tensor, ctx: StepContext, view, out: torch.Tensor) -> bool:
+        if self.identity or self._sparse(x):
+            return False
+        self._activations(x, self._route(x)[0], out)
+        return True
+
+    def _activations(self, x: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor) -> None:
+        """Every expert's activations times the token's weight for it, ``[T, F]`` (which may be a
+        column block of a wider buffer)."""
+        if self._project_fused(x, route_w, act):
+            return
+        ops.moe_act(linear(x, self.w_gate_up), route_w, act, self.E, self.ff,
+                    shared_gate=self.gated_shared, expert_act=self.expert_act)
+
+    def _project_fused(self, x: torch.Tensor, route_w: torch.Tensor, act: torch.Tensor) -> bool:
+        """The stacked gate/up product with the activation and the weighting in its epilogue, for
+        few token rows and for many; False, having done nothing, where those kernels do not
+        run."""
+        if not FUSE_EXPERTS or x.dtype != torch.bfloat16:
+            return False
+        a, T, err = self.expert_act, x.shape[0], ops.error_word(x.device)
+        consts = dict(activation=a.activation, limit=a.limit, slope=a.slope,
+                      up_offset=a.up_offset)
+        mixture = ops.Mixture(route_w, self.E, self.ff, self.gated_shared, a.shared_limit)
+        pair_from = pair_token_limit()
+        if pair_from and T >= pair_from and self.ff % 32 == 0:
+            return ops.gemm_bf16_pair(x, self.w_gate_up, act, err, gated=True, mixture=mixture,
+                                      **consts)
+        if T > swiglu_token_limit() or self.ff % 8 or self.F % 8:
+            return False
+        if self._gated_plan is None:
+            self._gated_plan = ops.gemm_swiglu_plan(self.F, x.shape[1], x.device) or False
+        plan = self._gated_plan
+        if not plan or plan[1] < FUSE_SWIGLU_FILL * ops.num_sms(x.device):
+            return False
+        return ops.gemm_bf16_swiglu(x, self.w_gate_up, act, err, plan[0], mixture=mixture,
+                                    **consts)
 
 
 register_ffn("moe", MoEFeedForward)

@@ -15,6 +15,7 @@ from ..config.specs import NormSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
 from .base import BuildEnv, Norm, ResidualStream, register_norm
+from .linear import linear_add_tanh
 
 
 class RMSNorm(Norm):
@@ -187,6 +188,12 @@ class TanhNorm(Norm):
             stream.pending = stream.pending_bias = None
             stream.reading = None
         return out
+
+    def fused_add_linear(self, x: torch.Tensor, d, assign: bool = False):
+        """The product ``d`` added into the stream ``x`` (``assign``: put in its place) and this
+        norm of the result, in one kernel; None where that kernel does not run."""
+        return linear_add_tanh(d.x, d.w, x, d.bias, self.alpha, self.weight, self.bias,
+                               assign=assign)
 
 
 register_norm("tanh_norm", TanhNorm)
