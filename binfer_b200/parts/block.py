@@ -7,7 +7,7 @@ the next norm, this layer's or the following one's.  A layer without a feed-forw
 """
 from __future__ import annotations
 
-from typing import List
+from typing import List, Optional
 
 from ..config.specs import LayerSpec, NameLayout
 from .base import (BuildEnv, EntryView, Part, ResidualStream, ScaledRows, StepContext, build_ffn,
@@ -34,6 +34,11 @@ class PreNormBlock(Part):
         return [part for part in (self.input_norm, self.mixer, self.post_norm, self.ffn)
                 if part is not None]
 
+    @property
+    def first_norm(self):
+        """The norm that reads the stream first."""
+        return self.input_norm
+
     def param_specs(self):
         return [s for part in self.parts() for s in part.param_specs()]
 
@@ -42,16 +47,14 @@ class PreNormBlock(Part):
             part.load(get)
 
     def forward(self, stream: ResidualStream, ctx: StepContext, view: EntryView,
-                successor: "PreNormBlock" = None) -> None:
+                successor: Optional[Part] = None) -> None:
         """``successor``: the block that runs next on this stream, if any; its input norm
         can then be prepared by this block's last product."""
         h = self._for(self.mixer, self.input_norm.forward(stream))
         deferred = getattr(self.mixer, "forward_deferred", None)
         if self.ffn is None:
-            nxt = successor if isinstance(successor, PreNormBlock) else None
             if deferred is not None:
-                stream.add_linear(deferred(h, ctx, view), nxt.input_norm if nxt else None,
-                                  nxt.mixer if nxt else None)
+                stream.add_linear(deferred(h, ctx, view), *self._reads_next(successor))
             else:
                 stream.add(self.mixer.forward(h, ctx, view))
             return
@@ -62,11 +65,16 @@ class PreNormBlock(Part):
         h = self._for(self.ffn, self.post_norm.forward(stream))
         deferred = getattr(self.ffn, "forward_deferred", None)
         if deferred is not None:
-            nxt = successor if isinstance(successor, PreNormBlock) else None
-            stream.add_linear(deferred(h, ctx), nxt.input_norm if nxt else None,
-                              nxt.mixer if nxt else None)
+            stream.add_linear(deferred(h, ctx), *self._reads_next(successor))
         else:
             stream.add(self.ffn.forward(h, ctx))
+
+    @staticmethod
+    def _reads_next(successor):
+        """The norm that reads the stream next, and the part that takes its output where that is
+        one part alone."""
+        return (getattr(successor, "first_norm", None),
+                successor.mixer if isinstance(successor, PreNormBlock) else None)
 
     @staticmethod
     def _for(part, h):

@@ -62,7 +62,7 @@ class ParallelBlock(Part):
             a.w_out, b.w_out = self.w_out[:, :a.out_cols], self.w_out[:, a.out_cols:]
 
     def forward(self, stream: ResidualStream, ctx: StepContext, view: EntryView,
-                successor: "ParallelBlock" = None) -> None:
+                successor: Optional[Part] = None) -> None:
         """``successor``: the block that runs next on this stream, if any; its norm can then be
         prepared by this block's last product."""
         h = stream.norm_input(self.norm)

@@ -96,9 +96,22 @@ class RMSNorm(Norm):
 register_norm("rmsnorm", RMSNorm)
 
 
-class LayerNorm(Norm):
+class _TwoDeltas(Norm):
+    """A norm whose kernel folds two pending adds."""
+
     takes_second_delta = True      # forward(..., also=): see ResidualStream.add_pair
 
+    @staticmethod
+    def _second_delta(stream: ResidualStream, also: Optional[torch.Tensor], rows):
+        """The second add, where the caller left it on the stream."""
+        if also is None and stream.pending2 is not None:
+            also = stream.pending2
+            if rows is None:
+                stream.pending2 = None
+        return also
+
+
+class LayerNorm(_TwoDeltas):
     """``y = (x - mean) / sqrt(var + eps) * w + b`` with the variance the mean of the squared
     deviations; the bias tensor is the weight's name with ``NormSpec.bias_suffix`` (None: no
     bias).  Folds the stream's pending add, and a second one (``also``), into the same pass."""
@@ -128,6 +141,7 @@ class LayerNorm(Norm):
         is).  ``also``: one more sublayer output to add beside the pending one."""
         if stream.pending_bias is not None:
             stream.flush()
+        also = self._second_delta(stream, also, rows)
         stream.ready = stream.ready_for = None
         n = n_rows if rows is not None else stream.x.shape[0]
         out = torch.empty((n, self.size), dtype=self.env.dtype, device=self.env.device)
@@ -142,12 +156,11 @@ class LayerNorm(Norm):
 register_norm("layernorm", LayerNorm)
 
 
-class TanhNorm(Norm):
+class TanhNorm(_TwoDeltas):
     """``y = tanh(alpha x) * w + b``: a norm that takes no statistic of the row (dynamic tanh);
     alpha is a tensor of one number.  Folds the stream's pending add, a second one (``also``)
     and the bias of the product that made them (``bias``) into the same pass."""
 
-    takes_second_delta = True      # forward(..., also=): see ResidualStream.add_pair
     takes_pending_bias = True      # ... and the stream's pending bias
 
     def __init__(self, spec: NormSpec, size: int, name: str, env: BuildEnv):
@@ -179,6 +192,7 @@ class TanhNorm(Norm):
         if rows is None and also is None and stream.ready_for is self:
             out, stream.ready, stream.ready_for = stream.ready, None, None
             return out           # the kernel before already prepared this norm
+        also = self._second_delta(stream, also, rows)
         stream.ready = stream.ready_for = None
         n = n_rows if rows is not None else stream.x.shape[0]
         out = torch.empty((n, self.size), dtype=self.env.dtype, device=self.env.device)

@@ -774,3 +774,110 @@ def make_pabelix_dir(tmp_path, which, dtype=torch.float32, raw=None, tweak=None,
         tweak(w)
     save_file(w, os.path.join(d, "model.safetensors"))
     return d
+
+
+# ------------------------------------------ the design whose looped passes project the stream
+def _naz_latent(heads, dim, rot_dim, vdim, rank, base=10000.0, scale=None, yarn=None):
+    rot = {"base": base, "dims": rot_dim}
+    if yarn is not None:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), yarn))
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank,
+            "rot": rot, "scale": (dim + rot_dim) ** -0.5 if scale is None else scale}
+
+
+def _naz_attn(heads, kv_heads, dim, vdim, window, rot_dims, base=10000.0, scale=None):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+            "mask": {"size": window}, "rot": {"base": base, "dims": rot_dims},
+            "scale": dim ** -0.5 if scale is None else scale}
+
+
+def _naz_dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def _naz_moe(experts, top, ff, limit, shared=None):
+    return {"kind": "moe", "router": {"experts": experts, "top": top},
+            "expert": {"ff": ff, "limit": limit},
+            "shared": None if shared is None else {"ff": shared[0], "limit": shared[1]}}
+
+
+def _naz_layer(kind, mixer, mlp=None):
+    return {"type": kind, "mixer": mixer, "mlp": mlp}
+
+
+# the loop from the first layer on, twice, a layer behind it; a window of 24; part of a head
+# turned; stretched waves; two limits; a layer without a feed-forward
+NAZ_A = {"architecture": "Nazorax", "vocab": 300, "width": 64, "norm": {"eps": 1e-5},
+         "loop": {"start": 0, "stop": 2, "times": 2},
+         "layers": [_naz_layer("attention", _naz_attn(4, 2, 32, 16, 24, 20, scale=0.3),
+                               _naz_dense(96)),
+                    _naz_layer("latent_attention",
+                               _naz_latent(3, 24, 8, 20, 40, scale=0.2, yarn=(4.0, 64, 8.0, 1.0)),
+                               _naz_moe(8, 2, 32, 1.5, (48, 0.7))),
+                    _naz_layer("latent_attention",
+                               _naz_latent(2, 16, 12, 28, 24, base=500.0, yarn=(2.5, 32, 4.0, 0.5)))]}
+# the loop in the middle, three times; plain waves; a key head for every query head and six
+# heads on one; windows of seven and of two; one expert of five without a shared one, all of
+# four with one; values larger and smaller than keys
+NAZ_B = {"architecture": "Nazorax", "vocab": 211, "width": 48, "norm": {"eps": 1e-6},
+         "loop": {"start": 1, "stop": 3, "times": 3},
+         "layers": [_naz_layer("latent_attention", _naz_latent(2, 16, 16, 16, 24), _naz_dense(40)),
+                    _naz_layer("attention", _naz_attn(3, 3, 24, 40, 7, 24, base=700.0),
+                               _naz_moe(5, 1, 40, 0.9)),
+                    _naz_layer("attention", _naz_attn(6, 1, 12, 8, 2, 4)),
+                    _naz_layer("latent_attention",
+                               _naz_latent(1, 8, 4, 40, 12, yarn=(3.0, 40, 6.0, 1.0)),
+                               _naz_moe(4, 4, 16, 2.0, (24, 1.2)))]}
+# odd sizes everywhere, no loop; one head, one expert; a window wider than the sequences
+NAZ_C = {"architecture": "Nazorax", "vocab": 131, "width": 51, "norm": {"eps": 1e-5},
+         "layers": [_naz_layer("latent_attention",
+                               _naz_latent(1, 9, 6, 7, 13, base=3000.0, yarn=(2.0, 16, 4.0, 1.0)),
+                               _naz_dense(13)),
+                    _naz_layer("attention", _naz_attn(1, 1, 7, 5, 400, 6), _naz_moe(1, 1, 11, 1.0)),
+                    _naz_layer("attention", _naz_attn(3, 3, 10, 6, 1, 2), _naz_moe(3, 2, 9, 0.5, (7, 0.8)))]}
+# wider, for bfloat16 and the tensor-core kernels; the whole model is the loop, walked once
+NAZ_D = {"architecture": "Nazorax", "vocab": 500, "width": 192, "norm": {"eps": 1e-5},
+         "loop": {"start": 0, "stop": 4, "times": 1},
+         "layers": [_naz_layer("latent_attention",
+                               _naz_latent(4, 64, 32, 64, 192, yarn=(4.0, 128, 16.0, 1.0)),
+                               _naz_dense(256)),
+                    _naz_layer("attention", _naz_attn(8, 4, 64, 64, 48, 64), _naz_moe(8, 2, 64, 2.0, (128, 1.0))),
+                    _naz_layer("latent_attention", _naz_latent(5, 32, 16, 48, 64),
+                               _naz_moe(4, 3, 96, 1.5)),
+                    _naz_layer("attention", _naz_attn(5, 5, 80, 112, 65, 40), _naz_dense(128))]}
+
+NAZ = {
+    "A": dict(raw=NAZ_A, std=0.08, norm_std=0.15, page_size=16, seed=55),
+    "B": dict(raw=NAZ_B, std=0.1, norm_std=0.15, page_size=4, seed=56),
+    "C": dict(raw=NAZ_C, std=0.12, norm_std=0.15, page_size=8, seed=57),
+    "D": dict(raw=NAZ_D, std=0.05, norm_std=0.1, page_size=16, seed=58),
+}
+
+
+def make_nazorax_dir(tmp_path, which, dtype=torch.float32, raw=None, tweak=None, tag="") -> str:
+    """A folder with config.json and random weights of a configuration of this design;
+    ``tweak(w)`` may change the tensors (a name -> tensor dictionary) before they are written."""
+    from binfer_b200.config import NazoraxConfig
+    from binfer_b200.parts.model import param_specs_for
+    from binfer_b200.weights import random_tensors, save_file
+    t = NAZ[which]
+    raw = raw or t["raw"]
+    cfg = NazoraxConfig.from_dict(raw)
+    d = os.path.join(str(tmp_path), f"naz_{which}{tag}_{str(dtype).split('.')[-1]}")
+    os.makedirs(d, exist_ok=True)
+    with open(os.path.join(d, "config.json"), "w") as f:
+        json.dump(cfg.to_dict(), f)
+    w = random_tensors(param_specs_for(cfg.to_spec()), t["seed"], t["std"], t["norm_std"], dtype)
+    for i, (n, x) in enumerate(sorted(w.items())):
+        if n == "embed":                 # of order one, so that the norms' tanh bends
+            x *= 0.8 / t["std"]
+        elif n.endswith(".alpha"):       # another one in every norm
+            x *= 0.4 + 0.3 * (i % 5)
+        elif n.endswith(".sink"):        # some of them above the scores
+            x *= 12.0
+        elif n.endswith((".gate", ".up", ".mix.q", ".mix.dkv")):
+            x *= 3.0                     # the clamps are reached now and then; sharper scores
+    if tweak is not None:
+        tweak(w)
+    save_file(w, os.path.join(d, "model.safetensors"))
+    return d
