@@ -373,13 +373,14 @@ def differential_config(size, layers=8):
 
 
 def projected_config(size, layers=8):
-    """The design whose looped passes project the stream, at the Qwen3 shape of that name,
-    ``layers`` layer runs (an even number): latent attention with a dense feed-forward, windowed
-    attention and latent attention with a mixture, walked ``(layers - 2) / 3`` times, then one more
-    of latent and of windowed attention for what is left.  Windowed attention has the shape's
-    heads and a window of 1,024, latent attention as many heads, of 128 plain and 64 rotated
-    sizes, over a latent of 512; the dense feed-forward is the shape's, the mixture eight experts
-    of which two run, which with the shared expert are as many active inner features."""
+    """The design whose looped passes project the stream, at the Qwen3 shape of that name, in
+    ``layers`` layer runs: three layers (latent attention with a dense feed-forward, windowed
+    attention with a mixture, latent attention with a mixture) walked ``(layers - 1) // 3`` times,
+    then latent and windowed attention with mixtures in turn for what is left.  Windowed attention
+    has the shape's heads and a window of 1,024, latent attention as many heads, of 128 plain and
+    64 rotated sizes, over a latent of 512; the dense feed-forward is the shape's, the mixture
+    eight experts of which two run, which with the shared expert are as many active inner
+    features."""
     width, heads, kv, d, ff = HYBRID_SIZES[size][:5]
     dense = {"kind": "dense", "ff": ff}
     moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0},

@@ -6,6 +6,9 @@
     python -m binfer_b200.microbench diff_decode --batch 8 --head-dim 64 --value-dim 128
     python -m binfer_b200.microbench gemm --tokens 8 --features 6144 --k 4096 [--library]
     python -m binfer_b200.microbench add_rmsnorm --tokens 8 --hidden 4096
+    python -m binfer_b200.microbench add_tanh_norm --tokens 2048 --hidden 4096
+    python -m binfer_b200.microbench experts --tokens 2048 --k 2048 --intermediate 6144
+    python -m binfer_b200.microbench out_product --tokens 8 --features 2048 --k 17408
     BINFER_B200_TRACE=1 python -m binfer_b200.microbench step_timeline --batch 8 --ctx 4096 --layers 6
 
 Sizes default to the Qwen3-8B shape.  Each kernel runs on a rotation of input sets
@@ -265,6 +268,91 @@ def add_rmsnorm(a):
     report("add_rmsnorm", us, nbytes=T * H * (4 + 4 + 2 + 2), tokens=T, hidden=H)
 
 
+def _stream_sets(a):
+    """(stream, pending output) pairs that together exceed the L2 cache."""
+    dev, T, H = torch.device("cuda:0"), a.tokens, a.hidden
+    sets = max(2, min(64, int(3e8 // (T * H * 6)) + 1))
+    return [(torch.randn(T, H, device=dev), torch.randn(T, H, device=dev).to(BF16))
+            for _ in range(sets)]
+
+
+def add_tanh_norm(a):
+    """The stream's pending add and bias with the tanh norm (--tokens, --hidden), beside
+    ``add_rmsnorm`` on the same rotation of inputs, and the pair that a pass starts from."""
+    T, H = a.tokens, a.hidden
+    sets = _stream_sets(a)
+    w, b = torch.ones(H, device="cuda:0"), torch.zeros(H, device="cuda:0")
+    out = torch.empty(T, H, device="cuda:0", dtype=BF16)
+    pair = torch.empty(T, 2 * H, device="cuda:0", dtype=BF16)
+    table = torch.randn(4096, H, device="cuda:0").to(BF16)
+    ids = torch.randint(0, 4096, (T,), device="cuda:0", dtype=torch.int32)
+    err = ops.error_word(torch.device("cuda:0"))
+    report("add_tanh_norm", timed([lambda x=x, d=d: ops.add_tanh_norm(
+        x, d, None, b, 0.5, w, b, out) for x, d in sets], a.iters, a.warmup),
+        nbytes=T * H * (4 + 4 + 2 + 2), tokens=T, hidden=H)
+    report("add_rmsnorm", timed([lambda x=x, d=d: ops.add_rmsnorm(x, d, w, out, 1e-6)
+                                 for x, d in sets], a.iters, a.warmup),
+           nbytes=T * H * (4 + 4 + 2 + 2), tokens=T, hidden=H)
+    report("stream_pair", timed([lambda x=x, d=d: ops.stream_pair(
+        x, d, None, b, table, ids, 1.0, pair, err) for x, d in sets], a.iters, a.warmup),
+        nbytes=T * H * (4 + 2 + 2 + 4), tokens=T, hidden=H)
+
+
+def out_product(a):
+    """The output product of few tokens with the stream's add and the tanh norm in its epilogue
+    (--tokens, --features, --k), beside the product alone and the norm behind it."""
+    dev = torch.device("cuda:0")
+    M, N, K = a.tokens, a.features, a.k
+    ws = [(0.05 * torch.randn(N, K, device=dev)).to(BF16)
+          for _ in range(max(2, int(3e8 // (N * K * 2)) + 1))]
+    x, resid = torch.randn(M, K, device=dev).to(BF16), torch.randn(M, N, device=dev)
+    nw, nb, err = torch.ones(N, device=dev), torch.zeros(N, device=dev), ops.error_word(dev)
+    y, out = torch.empty(M, N, device=dev, dtype=BF16), torch.empty(M, N, device=dev, dtype=BF16)
+    plan = ops.gemm_cluster_plan(N, K, dev)
+
+    def two(w):
+        ops.gemm_bf16_cluster(x, w, y, err, *plan)
+        ops.add_tanh_norm(resid, y, None, nb, 0.5, nw, nb, out)
+    for name, fn in (("gemm_bf16_cluster_add_tanh", lambda w: ops.gemm_bf16_cluster_add_tanh(
+            x, w, resid, nb, 0.5, nw, nb, err, *plan)),
+            ("gemm_bf16_cluster + add_tanh_norm", two),
+            ("gemm_bf16_cluster", lambda w: ops.gemm_bf16_cluster(x, w, y, err, *plan))):
+        report(name, timed([lambda w=w, fn=fn: fn(w) for w in ws], a.iters, a.warmup),
+               nbytes=(N * K + M * K) * 2 + M * N * 10, flops=2.0 * M * N * K, tokens=M, features=N, k=K)
+
+
+def experts(a):
+    """The stacked gate/up product of eight experts of --intermediate / 4 and a shared one of half
+    of --intermediate (--tokens, --k) with the clamped activation and the tokens' weights in its
+    epilogue, beside the library's product followed by ``moe_act``."""
+    dev = torch.device("cuda:0")
+    M, K, E, ff, sh = a.tokens, a.k, 8, a.intermediate // 4, a.intermediate // 2
+    F = E * ff + sh
+    ws = [(0.05 * torch.randn(2 * F, K, device=dev)).to(BF16)
+          for _ in range(max(2, int(3e8 // (4 * F * K)) + 1))]
+    x, err = torch.randn(M, K, device=dev).to(BF16), ops.error_word(dev)
+    rw = torch.rand(M, E, device=dev) * (torch.rand(M, E, device=dev) < 0.25)
+    act, gu = (torch.empty(M, n * F, device=dev, dtype=BF16) for n in (1, 2))
+    k = dict(activation="clamped", limit=7.0, slope=1.702, up_offset=1.0)
+    ea = ops.ExpertAct("clamped", 7.0, 7.0, 1.702, 1.0)
+    mix = ops.Mixture(rw, E, ff, False, 7.0)
+
+    def two(w):
+        torch.mm(x, w.t(), out=gu)
+        ops.moe_act(gu, rw, act, E, ff, shared_gate=False, expert_act=ea)
+    cases = [("library product + moe_act", two)]
+    plan = ops.gemm_swiglu_plan(F, K, dev) if M <= ops.CLUSTER_MAX_TOKENS else None
+    if plan:
+        cases.insert(0, ("gemm_bf16_swiglu(mixture)", lambda w: ops.gemm_bf16_swiglu(
+            x, w, act, err, plan[0], mixture=mix, **k)))
+    if M >= 64:
+        cases.insert(0, ("gemm_bf16_pair(mixture)", lambda w: ops.gemm_bf16_pair(
+            x, w, act, err, gated=True, mixture=mix, **k)))
+    for name, fn in cases:
+        report(name, timed([lambda w=w, fn=fn: fn(w) for w in ws], a.iters, a.warmup),
+               nbytes=(2 * F * K + M * K + M * F) * 2, flops=4.0 * M * F * K, tokens=M, inner=F, k=K)
+
+
 FP32_TFLOPS_NOMINAL = 148 * 128 * 2 * 1.965e9 / 1e12      # FMA lanes x 2 x the largest SM clock
 
 
@@ -385,7 +473,8 @@ def main(argv=None):
                                  formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("kernel", choices=["decode_attention", "prefill_attention", "gemm",
                                        "swiglu", "add_rmsnorm", "step_timeline", "scan",
-                                       "diff_decode", "diff_prefill"])
+                                       "diff_decode", "diff_prefill", "add_tanh_norm",
+                                       "out_product", "experts"])
     ap.add_argument("--iters", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--batch", type=int, default=8)
@@ -432,7 +521,8 @@ def main(argv=None):
     {"decode_attention": decode_attention, "prefill_attention": prefill_attention,
      "gemm": gemm, "swiglu": swiglu, "add_rmsnorm": add_rmsnorm,
      "step_timeline": step_timeline, "scan": scan, "diff_decode": diff_decode,
-     "diff_prefill": diff_prefill}[a.kernel](a)
+     "diff_prefill": diff_prefill, "add_tanh_norm": add_tanh_norm,
+     "out_product": out_product, "experts": experts}[a.kernel](a)
     return 0
 
 
