@@ -301,8 +301,8 @@ class LatentAttentionSpec:
     set by the mixer).  ``q_rank`` > 0: the queries go through a latent too, ``q = W_uq
     rmsnorm(W_dq h)`` with a weight of ``q_rank`` numbers (tensors ``dq``, ``dq_norm``, ``uq``
     in place of ``q``).  ``sinks``: a learned logit per head (tensor ``sink``) joins the
-    softmax's denominator; it has no key and no value and is not scaled.  ``names``: the tensors
-    inside the mixer's prefix."""
+    softmax's denominator as it is stored and brings no value.  ``names``: the tensors inside the
+    mixer's prefix."""
 
     kind: str = "latent_attention"
     num_heads: int = 0
