@@ -841,7 +841,7 @@ NAZ_D = {"architecture": "Nazorax", "vocab": 500, "width": 192, "norm": {"eps": 
          "layers": [_naz_layer("latent_attention",
                                _naz_latent(4, 64, 32, 64, 192, yarn=(4.0, 128, 16.0, 1.0)),
                                _naz_dense(256)),
-                    _naz_layer("attention", _naz_attn(8, 4, 64, 64, 48, 64), _naz_moe(8, 2, 64, 2.0, (128, 1.0))),
+                    _naz_layer("attention", _naz_attn(8, 4, 64, 64, 48, 64), _naz_moe(7, 2, 64, 1.8, (160, 0.9))),
                     _naz_layer("latent_attention", _naz_latent(5, 32, 16, 48, 64),
                                _naz_moe(4, 3, 96, 1.5)),
                     _naz_layer("attention", _naz_attn(5, 5, 80, 112, 65, 40), _naz_dense(128))]}

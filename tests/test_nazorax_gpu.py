@@ -275,7 +275,7 @@ def test_product_with_the_add_and_the_tanh_norm(cuda_device, tokens, N, K):
     assert int(err.item()) == 0
 
 
-@pytest.mark.parametrize("H_,rank,rot,ps", [(6, 96, 16, 16), (3, 16, 0, 8), (16, 512, 64, 16), (40, 48, 32, 64)])
+@pytest.mark.parametrize("H_,rank,rot,ps", [(7, 80, 32, 16), (3, 16, 0, 8), (16, 512, 64, 16), (40, 48, 32, 64)])
 def test_latent_attention_kernel_with_sinks(cuda_device, H_, rank, rot, ps):
     """The tensor-core kernel and its merge with a logit per head in the denominator: below, among
     and far above the scores; prompts, portions inside tiles, single tokens whose keys are shared
